@@ -44,6 +44,8 @@ class ScheduleEntry:
     cache: int
     owns_cache: bool = True
     kv_from: Optional[int] = None
+    junction: Optional[int] = None        # index into `ModelSpec.junctions`: what happens to the stream right before this run
+    turn: int = 0                         # which time that junction is passed (a loop's pass), counted from 0
 
 
 @dataclass(frozen=True)
@@ -61,6 +63,8 @@ class ModelSpec:
     embed_scale: Optional[float] = None   # factor on the embedding rows (None: 1)
     logit_cap: Optional[float] = None     # soft cap on the logits, cap * tanh(logits / cap) (None: none)
     embedding: Optional[PartSpec] = None  # what is added to the token embedding (a part of `parts.EMBEDDINGS`; None: nothing)
+    junctions: List[PartSpec] = field(default_factory=list)   # parts of `parts.JUNCTIONS` that schedule entries name
+    token_table: int = 0                  # columns of the per-token side table that layers' token inputs read (0: none)
     launch_overlap: bool = True           # kernels of a step may start while their predecessor drains; False: strictly in turn
 
     def validate(self) -> None:
@@ -72,6 +76,8 @@ class ModelSpec:
         for i, e in enumerate(self.schedule):
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule[{i}] names layer {e.layer}, the model has {len(self.layers)}")
+            if e.junction is not None and not 0 <= e.junction < len(self.junctions):
+                raise ValueError(f"schedule[{i}] names junction {e.junction}, the model has {len(self.junctions)}")
             if e.owns_cache:
                 if e.cache in owners:
                     raise ValueError(f"cache entry {e.cache} has two owners: schedule[{owners[e.cache]}] and [{i}]")

@@ -39,6 +39,7 @@ LIBRARIES = {
     "latent": (["latent.cu"], [], []),
     "recurrent": (["recurrent.cu"], [], []),
     "moe": (["moe.cu"], [], []),
+    "gla": (["gla.cu"], [], []),
 }
 HEADERS = ["common.cuh", "attn_decode_noalloc.h"]
 

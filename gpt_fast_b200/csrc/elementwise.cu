@@ -2,7 +2,9 @@
 // (erf) GELU, the tanh form of GELU, SiLU, and the square of ReLU.  Arithmetic is 32-bit.  Products apply the same
 // functions in their epilogue where they can; this kernel serves the shapes that cannot.
 // Also a sigmoid gate on the columns of a tensor, one gate per group of columns (a head, or a single column), and the
-// last step of differential attention: the difference of a head's two maps, normed over the head.
+// last step of differential attention: the difference of a head's two maps, normed over the head.  And the entry of a
+// pass of a loop of layers: the stream beside the embedding output as the input of a product, the stream itself replaced by
+// the pass's vector, to which the product is added.
 #include "common.cuh"
 
 GFB_DEFINE_LAST_ERROR()
@@ -95,4 +97,36 @@ GFB_API int gfb_diff_combine(const void* a, void* out, int dt, int T, int H, int
     else if (dt == GFB_F32) e = gfb_launch(diff_combine_kernel<float>, dim3(blocks), dim3(128), 0, stream, (const float*)a, (float*)out, items, dv, lambda, eps, out_scale);
     else return gfb_fail("gfb_diff_combine: unknown type %d", dt);
     return gfb_check(e, "gfb_diff_combine");
+}
+
+// cat[t] = [x[t] ; x0[t]] in the compute type, y[t] = step; 32-bit rows of D numbers
+template <typename TO, typename TS>
+__global__ void __launch_bounds__(256)
+pass_entry_kernel(const float* __restrict__ x, const float* __restrict__ x0, const TS* __restrict__ step, TO* __restrict__ cat,
+                  float* __restrict__ y, int D, size_t n) {
+    gfb_pdl_launch();
+    gfb_pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const size_t t = i / D;
+    const int c = (int)(i - t * D);
+    cat[2 * t * D + c] = gfb_from_f32<TO>(x[i]);
+    cat[(2 * t + 1) * D + c] = gfb_from_f32<TO>(x0[i]);
+    y[i] = gfb_to_f32(step[c]);
+}
+
+// x, x0, y float32 [T, D] (y is not x or x0), step [D] of type step_dt, cat [T, 2 D] of type cat_dt
+GFB_API int gfb_pass_entry(const float* x, const float* x0, const void* step, int step_dt, void* cat, int cat_dt, float* y, int T, int D,
+                           cudaStream_t stream) {
+    const size_t n = (size_t)T * D;
+    if (n == 0) return 0;
+    const unsigned blocks = (unsigned)((n + 255) / 256);
+    cudaError_t e;
+#define GO(TO, TS) e = gfb_launch(pass_entry_kernel<TO, TS>, dim3(blocks), dim3(256), 0, stream, x, x0, (const TS*)step, (TO*)cat, y, D, n)
+    if (cat_dt == GFB_BF16 && step_dt == GFB_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+    else if (cat_dt == GFB_BF16 && step_dt == GFB_F32) GO(__nv_bfloat16, float);
+    else if (cat_dt == GFB_F32 && step_dt == GFB_F32) GO(float, float);
+    else return gfb_fail("gfb_pass_entry: unsupported types %d and %d", cat_dt, step_dt);
+#undef GO
+    return gfb_check(e, "gfb_pass_entry");
 }

@@ -9,6 +9,9 @@
 //
 // And token embedding plus a learned vector per position: out[t] = table[tok_t] * scale + positions[p_t], p_t the
 // token's place in its sequence.
+//
+// And what a layer reads of a per-token side table: act[t, j] = gelu_tanh(z[t, j]) * side[tok_t][off + j], j < n, the layer's
+// n columns of the table starting at off.
 #include "common.cuh"
 
 GFB_DEFINE_LAST_ERROR()
@@ -115,4 +118,41 @@ GFB_API int gfb_embed_positions(const int* tokens, const void* table, const void
     else
         return gfb_fail("gfb_embed_positions: unknown table type %d", table_dt);
     return gfb_check(e, "gfb_embed_positions");
+}
+
+template <typename TW, typename TO>
+__global__ void __launch_bounds__(256)
+token_gate_kernel(const int* __restrict__ tokens, const TW* __restrict__ side, int ld_side, int off, const float* __restrict__ z,
+                  TO* __restrict__ out, int n, int V, size_t total, int* status) {
+    gfb_pdl_launch();
+    gfb_pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const int t = (int)(i / n), j = (int)(i - (size_t)t * n);
+    const int id = tokens[t];
+    if (id < 0 || id >= V) {
+        if (j == 0) gfb_report(status, GFB_ERR_TOKEN_RANGE, t, id);
+        out[i] = gfb_from_f32<TO>(0.f);
+        return;
+    }
+    const float v = z[i];
+    const float g = 0.5f * v * (1.0f + tanhf(0.79788456080286535588f * (v + 0.044715f * v * v * v)));
+    out[i] = gfb_from_f32<TO>(g * gfb_to_f32(side[(size_t)id * ld_side + off + j]));
+}
+
+// tokens int32 [T]; side [V, ld_side] of type side_dt, columns off .. off + n - 1; z float32 [T, n]; out [T, n] of type out_dt.
+GFB_API int gfb_token_gate(const int* tokens, const void* side, int side_dt, int V, int ld_side, int off, const float* z, void* out,
+                           int out_dt, int T, int n, int* status, cudaStream_t stream) {
+    const size_t total = (size_t)T * n;
+    if (total == 0) return 0;
+    if (off < 0 || off + n > ld_side) return gfb_fail("gfb_token_gate: columns %d .. %d of a table of %d", off, off + n - 1, ld_side);
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    cudaError_t e;
+#define GO(TW, TO) e = gfb_launch(token_gate_kernel<TW, TO>, dim3(blocks), dim3(256), 0, stream, tokens, (const TW*)side, ld_side, off, z, \
+                                  (TO*)out, n, V, total, status)
+    if (side_dt == GFB_BF16 && out_dt == GFB_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+    else if (side_dt == GFB_F32 && out_dt == GFB_F32) GO(float, float);
+    else return gfb_fail("gfb_token_gate: unsupported types %d and %d", side_dt, out_dt);
+#undef GO
+    return gfb_check(e, "gfb_token_gate");
 }

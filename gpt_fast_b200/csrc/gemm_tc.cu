@@ -1366,8 +1366,8 @@ GFB_API int gfb_gemm_tc(const void* A, const void* W, void* out, int out_dt, int
 // (rows a multiple of tile_rows), W [groups, N, K].  tile_rows 16, 32, 64: the swapped orientation of a decode step (128 weight
 // rows x a tile of tokens per block); 128: 128 tokens x 128 or 64 weight rows per block; in both a tile whose entry is negative is
 // skipped.  tile_rows 256: pairs of SMs walk over the first *tiles_used row tiles (the entries with rows come first).
-// epi: EPI_STORE with out float32 [rows, N], or EPI_GLU_CLAMP with out bfloat16 [rows, N / 2] from alternating gate/up
-// rows of W.
+// epi: EPI_STORE with out float32 [rows, N], EPI_GLU_CLAMP with out bfloat16 [rows, N / 2] from alternating gate/up
+// rows of W, or EPI_RELU2 with out bfloat16 [rows, N].
 GFB_API int gfb_gemm_tc_grouped(const void* A, const void* W, void* out, int out_dt, int rows, int tile_rows, int groups, int N, int K,
                                 int epi, const int* tile_group, const int* tiles_used, float limit, float alpha, float shift,
                                 int* status, cudaStream_t stream) {
@@ -1390,10 +1390,12 @@ GFB_API int gfb_gemm_tc_grouped(const void* A, const void* W, void* out, int out
         if (make_map(&mx, W, groups * N, K, BM)) return 1;
         if (make_map(&my, A, rows, K, tile_rows)) return 1;
         const bool glu = epi == EPI_GLU_CLAMP && out_dt == GFB_BF16, store = epi == EPI_STORE && out_dt == GFB_F32;
+        const bool relu2 = epi == EPI_RELU2 && out_dt == GFB_BF16;
         const int ldo = glu ? N / 2 : N;
-#define GS(B) return glu ? launch_grouped<B, EPI_GLU_CLAMP, __nv_bfloat16, true>(mx, my, out, N, rows, K, ldo, STAGES, status, gp, stream) \
+#define GS(B) return relu2 ? launch_grouped<B, EPI_RELU2, __nv_bfloat16, true>(mx, my, out, N, rows, K, ldo, STAGES, status, gp, stream) \
+                         : glu ? launch_grouped<B, EPI_GLU_CLAMP, __nv_bfloat16, true>(mx, my, out, N, rows, K, ldo, STAGES, status, gp, stream) \
                          : launch_grouped<B, EPI_STORE, float, true>(mx, my, out, N, rows, K, ldo, STAGES, status, gp, stream)
-        if (glu || store) {
+        if (glu || store || relu2) {
             if (tile_rows == 16) GS(16);
             if (tile_rows == 32) GS(32);
             GS(64);
@@ -1406,6 +1408,8 @@ GFB_API int gfb_gemm_tc_grouped(const void* A, const void* W, void* out, int out
         if (make_map(&my, W, groups * N, K, 128)) return 1;
         if (epi == EPI_GLU_CLAMP && out_dt == GFB_BF16)
             return launch_pair_grouped<EPI_GLU_CLAMP, __nv_bfloat16>(mx, my, out, rows, N, K, N / 2, status, gp, stream);
+        if (epi == EPI_RELU2 && out_dt == GFB_BF16)
+            return launch_pair_grouped<EPI_RELU2, __nv_bfloat16>(mx, my, out, rows, N, K, N, status, gp, stream);
         if (epi == EPI_STORE && out_dt == GFB_F32)
             return launch_pair_grouped<EPI_STORE, float>(mx, my, out, rows, N, K, N, status, gp, stream);
         return gfb_fail("gfb_gemm_tc_grouped: unsupported epilogue %d / output type %d", epi, out_dt);
@@ -1418,6 +1422,9 @@ GFB_API int gfb_gemm_tc_grouped(const void* A, const void* W, void* out, int out
     if (epi == EPI_GLU_CLAMP && out_dt == GFB_BF16)
         return narrow ? launch_grouped<64, EPI_GLU_CLAMP, __nv_bfloat16>(mx, my, out, rows, N, K, N / 2, STAGES, status, gp, stream)
                       : launch_grouped<128, EPI_GLU_CLAMP, __nv_bfloat16>(mx, my, out, rows, N, K, N / 2, STAGES, status, gp, stream);
+    if (epi == EPI_RELU2 && out_dt == GFB_BF16)
+        return narrow ? launch_grouped<64, EPI_RELU2, __nv_bfloat16>(mx, my, out, rows, N, K, N, STAGES, status, gp, stream)
+                      : launch_grouped<128, EPI_RELU2, __nv_bfloat16>(mx, my, out, rows, N, K, N, STAGES, status, gp, stream);
     if (epi == EPI_STORE && out_dt == GFB_F32)
         return narrow ? launch_grouped<64, EPI_STORE, float>(mx, my, out, rows, N, K, N, STAGES, status, gp, stream)
                       : launch_grouped<128, EPI_STORE, float>(mx, my, out, rows, N, K, N, STAGES, status, gp, stream);

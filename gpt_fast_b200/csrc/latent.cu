@@ -10,8 +10,10 @@
 //                      `rot` outputs rotated by the token's position; both appended to the cache as one row;
 //                      every head's rotated query part turned and written behind the head's latent query.
 // gfb_headwise_linear  out[t, h, :] = in[t, h, :] W_h with a weight per head (the two expansions above), strided
-//                      inputs and outputs, optionally times sigmoid(gate[t, h, :]).
-// gfb_latent_attention attention on the cached rows for bfloat16 on tensor cores (below).
+//                      inputs and outputs, optionally times sigmoid(gate[t, h, :]), or times sigmoid(gate[t, h]) with one
+//                      gate per head.
+// gfb_latent_attention attention on the cached rows for bfloat16 on tensor cores (below), optionally over a sliding window
+//                      and with a sink per head.
 // Norm, angles and rotation are 32-bit; sums are 32-bit in a fixed order.
 #include "common.cuh"
 
@@ -141,7 +143,7 @@ constexpr int HT_ROWS = 64, HT_COLS = 64, HT_K = 64, HT_PAD = 8;
 __global__ void __launch_bounds__(128)
 headwise_linear_tc_kernel(const __nv_bfloat16* __restrict__ in, int ld_in, int in_off, int in_stride, const __nv_bfloat16* __restrict__ w,
                           __nv_bfloat16* __restrict__ out, int ld_out, int out_off, int out_stride, const __nv_bfloat16* __restrict__ gate,
-                          int ld_gate, int gate_off, int n_tokens, int K, int N) {
+                          int ld_gate, int gate_off, int gate_cols, int n_tokens, int K, int N) {
     __shared__ __align__(16) __nv_bfloat16 sA[HT_ROWS][HT_K + HT_PAD];
     __shared__ __align__(16) __nv_bfloat16 sW[HT_K][HT_COLS + HT_PAD];
     gfb_pdl_launch();
@@ -189,7 +191,7 @@ headwise_linear_tc_kernel(const __nv_bfloat16* __restrict__ in, int ld_in, int i
             const int t = r0 + 8 * (e >> 1), n = n0 + j * 8 + 2 * (lane & 3) + (e & 1);
             if (t < n_tokens && n < N) {
                 float v = acc[j][e];
-                if (gate != nullptr) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * ld_gate + gate_off + (size_t)h * N + n])));
+                if (gate != nullptr) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * ld_gate + gate_off + (gate_cols == 1 ? (size_t)h : (size_t)h * N + n)])));
                 out[(size_t)t * ld_out + out_off + (size_t)h * out_stride + n] = __float2bfloat16_rn(v);
             }
         }
@@ -210,7 +212,7 @@ template <typename T>
 __global__ void __launch_bounds__(HL_THREADS)
 headwise_linear_kernel(const T* __restrict__ in, int ld_in, int in_off, int in_stride, const T* __restrict__ w,
                        T* __restrict__ out, int ld_out, int out_off, int out_stride, const T* __restrict__ gate, int ld_gate,
-                       int gate_off, int n_tokens, int K, int N) {
+                       int gate_off, int gate_cols, int n_tokens, int K, int N) {
     extern __shared__ float xs[];                 // [HL_TT][K], then [HL_KS][HL_TT][HL_COLS] partial sums
     float* part = xs + (size_t)HL_TT * K;
     gfb_pdl_launch();
@@ -246,16 +248,17 @@ headwise_linear_kernel(const T* __restrict__ in, int ld_in, int in_off, int in_s
         float v = part[(size_t)tt * HL_COLS + cc];
 #pragma unroll
         for (int s = 1; s < HL_KS; s++) v += part[((size_t)s * HL_TT + tt) * HL_COLS + cc];
-        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-gfb_to_f32(gate[(size_t)(t0 + tt) * ld_gate + gate_off + (size_t)h * N + col])));
+        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-gfb_to_f32(gate[(size_t)(t0 + tt) * ld_gate + gate_off + (gate_cols == 1 ? (size_t)h : (size_t)h * N + col)])));
         out[(size_t)(t0 + tt) * ld_out + out_off + (size_t)h * out_stride + col] = gfb_from_f32<T>(v);
     }
 }
 
 // in [T, ld_in]: head h's K inputs start at column in_off + h * in_stride; out [T, ld_out] likewise; w [H, K, N]; gate (or
-// null) [T, ld_gate] with head h's N gate values at column gate_off + h * N.  One type for all.
+// null) [T, ld_gate] with head h's N gate values at column gate_off + h * N, or (gate_cols = 1) its one gate at gate_off + h.
+// One type for all.
 GFB_API int gfb_headwise_linear(const void* in, int dt, int ld_in, int in_off, int in_stride, const void* w, void* out,
                                 int ld_out, int out_off, int out_stride, const void* gate, int ld_gate, int gate_off,
-                                int n_tokens, int H, int K, int N, cudaStream_t stream) {
+                                int gate_cols, int n_tokens, int H, int K, int N, cudaStream_t stream) {
     if (n_tokens <= 0 || H <= 0 || N <= 0) return 0;
     if (K <= 0) return gfb_fail("gfb_headwise_linear: K = %d", K);
     if (H > 65535 || (N + HL_COLS - 1) / HL_COLS > 65535) return gfb_fail("gfb_headwise_linear: %d heads of %d columns exceed the grid limit", H, N);
@@ -264,7 +267,7 @@ GFB_API int gfb_headwise_linear(const void* in, int dt, int ld_in, int in_off, i
         dim3 grid((n_tokens + HT_ROWS - 1) / HT_ROWS, H, (N + HT_COLS - 1) / HT_COLS);
         cudaError_t e = gfb_launch(headwise_linear_tc_kernel, grid, dim3(128), 0, stream, (const __nv_bfloat16*)in, ld_in, in_off, in_stride,
                                    (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ld_out, out_off, out_stride, (const __nv_bfloat16*)gate,
-                                   ld_gate, gate_off, n_tokens, K, N);
+                                   ld_gate, gate_off, gate_cols, n_tokens, K, N);
         return gfb_check(e, "gfb_headwise_linear (tensor cores)");
     }
     const size_t smem = ((size_t)HL_TT * K + (size_t)HL_KS * HL_TT * HL_COLS) * sizeof(float);
@@ -279,7 +282,7 @@ GFB_API int gfb_headwise_linear(const void* in, int dt, int ld_in, int in_off, i
             allowed = 160 * 1024;                                                                                           \
         }                                                                                                                   \
         e = gfb_launch(headwise_linear_kernel<T>, grid, dim3(HL_THREADS), smem, stream, (const T*)in, ld_in, in_off, in_stride, \
-                       (const T*)w, (T*)out, ld_out, out_off, out_stride, (const T*)gate, ld_gate, gate_off, n_tokens, K, N); \
+                       (const T*)w, (T*)out, ld_out, out_off, out_stride, (const T*)gate, ld_gate, gate_off, gate_cols, n_tokens, K, N); \
     } while (0)
     if (dt == GFB_BF16) GO(__nv_bfloat16);
     else if (dt == GFB_F32) GO(float);
@@ -296,7 +299,9 @@ GFB_API int gfb_headwise_linear(const void* in, int dt, int ld_in, int in_off, i
 // each scores half of the tile's keys, they agree on the rows' maxima and exchange their softmax weights through shared
 // memory (two barriers of 64 threads per tile), and each keeps half of the value columns of O in registers (128 numbers
 // per thread at rank 512).  bfloat16 operands on `mma.sync.m16n8k16`, scores, softmax and sums in 32-bit; the softmax
-// weights are rounded to bfloat16 for the second product.  Keys are masked per row by the row's own position.
+// weights are rounded to bfloat16 for the second product.  Keys are masked per row by the row's own position and, with a
+// window, by the distance to it; a block starts at the first tile that its earliest row sees.  A sink adds exp(sink_h) to
+// a row's denominator (behind the last tile, or where the slices are combined).
 constexpr int LA_ROWS = 64;           // query rows per block
 constexpr int LA_KEYS = 32;           // cached rows per tile
 constexpr int LA_THREADS = 256;
@@ -306,7 +311,8 @@ constexpr int LA_PAD = 8;             // bfloat16 numbers of padding per shared-
 template <int NT>
 __global__ void __launch_bounds__(LA_THREADS, 1)
 latent_attention_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, GfbPagedKV kv, GfbBatch b,
-                        int H, int Dk, int R, float scale_log2, int n_splits, float* __restrict__ partial, int* status) {
+                        int H, int Dk, int R, float scale_log2, int window, const float* __restrict__ sink, int n_splits,
+                        float* __restrict__ partial, int* status) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int DkP = Dk + LA_PAD;
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem_raw);            // [LA_ROWS][DkP]
@@ -324,9 +330,10 @@ latent_attention_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __re
     const int rows_here = min(LA_ROWS, n_rows - m0);
     const int last_pos = start + (m0 + rows_here - 1) / H;                      // the latest position any row of the block sees
     const int all_tiles = last_pos / LA_KEYS + 1;
+    const int first_tile = window > 0 ? max(0, start + m0 / H - window + 1) / LA_KEYS : 0;      // the first tile the earliest row sees
     // with n_splits > 1 (a decode step) the block takes one slice of the cached rows and leaves its unnormalised sums
-    const int per_split = (all_tiles + n_splits - 1) / n_splits;
-    const int tile_lo = blockIdx.z * per_split, n_tiles = min(all_tiles, tile_lo + per_split);
+    const int per_split = (all_tiles - first_tile + n_splits - 1) / n_splits;
+    const int tile_lo = first_tile + blockIdx.z * per_split, n_tiles = min(all_tiles, tile_lo + per_split);
     const int* pt = kv.page_table + (size_t)slot * kv.max_pages;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int chunks = Dk / 8;                                                  // 16-byte pieces of a row
@@ -363,6 +370,8 @@ latent_attention_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __re
     const int nt_all = R / 8, nt_lo = half == 0 ? 0 : (nt_all + 1) / 2, nt_n = half == 0 ? (nt_all + 1) / 2 : nt_all - (nt_all + 1) / 2;
     const int r0 = rw + (lane >> 2);                   // rows of this thread's accumulator values: r0 and r0 + 8
     const int pos0 = (r0 < rows_here) ? start + (m0 + r0) / H : -1, pos1 = (r0 + 8 < rows_here) ? start + (m0 + r0 + 8) / H : -1;
+    // the first key each row sees (no window: all of them)
+    const int lo0 = window > 0 ? pos0 - window + 1 : 0, lo1 = window > 0 ? pos1 - window + 1 : 0;
     float o[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
@@ -398,8 +407,8 @@ latent_attention_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __re
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int key = key0 + j * 8 + e;
-                sc[j][e] = key <= pos0 ? sc[j][e] * scale_log2 : -INFINITY;
-                sc[j][2 + e] = key <= pos1 ? sc[j][2 + e] * scale_log2 : -INFINITY;
+                sc[j][e] = key <= pos0 && key >= lo0 ? sc[j][e] * scale_log2 : -INFINITY;
+                sc[j][2 + e] = key <= pos1 && key >= lo1 ? sc[j][2 + e] * scale_log2 : -INFINITY;
                 t0m = fmaxf(t0m, sc[j][e]);
                 t1m = fmaxf(t1m, sc[j][2 + e]);
             }
@@ -481,7 +490,18 @@ latent_attention_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __re
         }
         return;
     }
-    const float i0 = l0 > 0.f ? 1.0f / l0 : 0.f, i1 = l1 > 0.f ? 1.0f / l1 : 0.f;
+    float i0, i1;
+    if (sink != nullptr) {
+        // o and l are relative to 2^mx; the sink may be the largest term of the row
+        const float k0 = sink[(m0 + r0) % H] * 1.4426950408889634f, k1 = sink[(m0 + r0 + 8) % H] * 1.4426950408889634f;
+        const float f0 = fmaxf(mx0, k0), f1 = fmaxf(mx1, k1);
+        const float c0 = exp2f(mx0 - f0), c1 = exp2f(mx1 - f1);
+        i0 = c0 / (l0 * c0 + exp2f(k0 - f0));
+        i1 = c1 / (l1 * c1 + exp2f(k1 - f1));
+    } else {
+        i0 = l0 > 0.f ? 1.0f / l0 : 0.f;
+        i1 = l1 > 0.f ? 1.0f / l1 : 0.f;
+    }
     __nv_bfloat16* orow = out + ((size_t)t0 * H + m0) * R;
 #pragma unroll
     for (int j = 0; j < NT; j++) {
@@ -493,8 +513,10 @@ latent_attention_kernel(const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __re
     }
 }
 
-// The slices of a row: out = sum_s O_s 2^(m_s - M) / sum_s l_s 2^(m_s - M), M the largest m_s, slices in ascending order.
-__global__ void latent_combine_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ out, int n_splits, int R) {
+// The slices of a row: out = sum_s O_s 2^(m_s - M) / (sum_s l_s 2^(m_s - M) + 2^(sink - M)), M the largest m_s (and the
+// sink, if there is one), slices in ascending order.
+__global__ void latent_combine_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ out, int n_splits, int R,
+                                      const float* __restrict__ sink, int H) {
     gfb_pdl_launch();
     gfb_pdl_wait();
     const size_t row = blockIdx.x;
@@ -502,6 +524,11 @@ __global__ void latent_combine_kernel(const float* __restrict__ partial, __nv_bf
     float M = -INFINITY;
     for (int s = 0; s < n_splits; s++) M = fmaxf(M, base[(size_t)s * (R + 2) + R]);
     float l = 0.f;
+    if (sink != nullptr) {
+        const float k = sink[row % H] * 1.4426950408889634f;
+        M = fmaxf(M, k);
+        l = exp2f(k - M);
+    }
     for (int s = 0; s < n_splits; s++) {
         const float m = base[(size_t)s * (R + 2) + R];
         if (m != -INFINITY) l += base[(size_t)s * (R + 2) + R + 1] * exp2f(m - M);
@@ -518,13 +545,14 @@ __global__ void latent_combine_kernel(const float* __restrict__ partial, __nv_bf
 }
 
 // q bfloat16 [T, H, Dk] (Dk = rank + rot), out bfloat16 [T, H * rank]; the cache entry holds one row of Dk numbers per
-// token in pages of a multiple of 32 tokens.  Needs Dk % 16 == 0, rank % 16 == 0, rank <= 512, rank < Dk.  n_splits > 1:
+// token in pages of a multiple of 32 tokens.  window > 0: a row sees that many latest positions, its own among them; sink
+// float32 [H] or null.  Needs Dk % 16 == 0, rank % 16 == 0, rank <= 512, rank < Dk.  n_splits > 1:
 // every sequence's cached rows are cut into that many slices with a block each, whose sums go through `partial`
 // (float32 [T * H, n_splits, rank + 2]) and a second kernel.
 GFB_API int gfb_latent_attention(const void* q, void* out, void* k_pool, const int* page_table, int max_pages, int page_size,
                                  int n_pages, const int* cu_seqlens, const int* tok_seq, const int* slots, const int* lengths,
-                                 int n_seqs, int n_tokens, int max_q_len, int H, int Dk, int R, float scale, int n_splits,
-                                 float* partial, int* status, cudaStream_t stream) {
+                                 int n_seqs, int n_tokens, int max_q_len, int H, int Dk, int R, float scale, int window,
+                                 const float* sink, int n_splits, float* partial, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (Dk % 16 || R % 16 || R > 512 || R >= Dk || page_size % LA_KEYS)
         return gfb_fail("gfb_latent_attention: rows of %d with %d value columns in pages of %d do not fit the kernel", Dk, R, page_size);
@@ -546,7 +574,7 @@ GFB_API int gfb_latent_attention(const void* q, void* out, void* k_pool, const i
         e = cudaFuncSetAttribute(latent_attention_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
         if (e != cudaSuccess) return gfb_fail("gfb_latent_attention: %s", cudaGetErrorString(e));                           \
         e = gfb_launch(latent_attention_kernel<NT>, grid, dim3(LA_THREADS), smem, stream, (const __nv_bfloat16*)q,          \
-                       (__nv_bfloat16*)out, kv, b, H, Dk, R, scale_log2, n_splits, partial, status);                        \
+                       (__nv_bfloat16*)out, kv, b, H, Dk, R, scale_log2, window, sink, n_splits, partial, status);                        \
     } while (0)
     if (nt <= 8) GO(8);
     else if (nt <= 16) GO(16);
@@ -555,6 +583,6 @@ GFB_API int gfb_latent_attention(const void* q, void* out, void* k_pool, const i
     if (gfb_check(e, "gfb_latent_attention")) return 1;
     if (n_splits == 1) return 0;
     e = gfb_launch(latent_combine_kernel, dim3((unsigned)n_tokens * H), dim3(128), 0, stream, (const float*)partial, (__nv_bfloat16*)out,
-                   n_splits, R);
+                   n_splits, R, sink, H);
     return gfb_check(e, "gfb_latent_attention (combine)");
 }

@@ -257,14 +257,15 @@ GFB_API int gfb_layernorm(float* x, const float* y, int S, long slice, const voi
 //                                           product split over K (added in ascending order), each with a
 //                                           per-column factor s_b (or none); written back
 //   (2) out_k[r] = (x - mean) / sqrt(var + eps_k) * w_k      up to two outputs from ONE mean and variance
-// The row sits in shared memory; statistics are 32-bit, the variance is the mean of squared deviations.
+// The row sits in shared memory, or in registers where its length allows 16-byte accesses (`layernorm_multi_vec_kernel`);
+// statistics are 32-bit, the variance is the mean of squared deviations.
 struct LnBranch {
     const float* y;      // [max(S, 1)][T][D], or null
     int S;
     const void* scale;   // [D] of type scale_dt, or null
 };
 struct LnOut {
-    const void* w;       // [D] of type w_dt
+    const void* w;       // [D] of type w_dt, or null: the row itself in the output's type, no norm
     float eps;
     void* out;           // [R][D], or null
 };
@@ -296,6 +297,11 @@ __global__ void layernorm_multi_kernel(float* __restrict__ x, LnBranch b0, LnBra
     }
     if (o0.out == nullptr && o1.out == nullptr) return;
     __syncthreads();
+    if (o0.out != nullptr && o0.w == nullptr) {                // the row as it is (the only output)
+        TO* o = (TO*)o0.out + (size_t)r * D;
+        for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = gfb_from_f32<TO>(row[i]);
+        return;
+    }
     float mean = 0.f;
     if (!rms) {
         float s = 0.f;
@@ -317,9 +323,118 @@ __global__ void layernorm_multi_kernel(float* __restrict__ x, LnBranch b0, LnBra
     }
 }
 
+// The same with the row in registers (NV float4 per thread), every branch's partial sums added in ascending order as above.
+template <int NV>
+__device__ __forceinline__ void add_branch(float4 (&v)[NV], const LnBranch& b, int scale_dt, size_t slice, size_t base, int nvec) {
+    float4 u[NV];
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        u[k] = i < nvec ? reinterpret_cast<const float4*>(b.y + base)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    constexpr int W = 8 / NV;                                // partial sums whose loads are in flight together
+    for (int p = 1; p < b.S; p += W) {
+        float4 a[W][NV];
+#pragma unroll
+        for (int q = 0; q < W; q++) {
+            const float4* pr = reinterpret_cast<const float4*>(b.y + (size_t)min(p + q, b.S - 1) * slice + base);
+#pragma unroll
+            for (int k = 0; k < NV; k++) {
+                const int i = threadIdx.x + k * blockDim.x;
+                a[q][k] = i < nvec ? pr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
+#pragma unroll
+        for (int q = 0; q < W; q++)
+            if (p + q < b.S) {
+#pragma unroll
+                for (int k = 0; k < NV; k++) { u[k].x += a[q][k].x; u[k].y += a[q][k].y; u[k].z += a[q][k].z; u[k].w += a[q][k].w; }
+            }
+    }
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (i < nvec) {
+            const float4 g = b.scale != nullptr ? ld_w4(b.scale, scale_dt, i) : make_float4(1.f, 1.f, 1.f, 1.f);
+            v[k].x += g.x * u[k].x; v[k].y += g.y * u[k].y; v[k].z += g.z * u[k].z; v[k].w += g.w * u[k].w;
+        }
+    }
+}
+
+template <typename TO, int NV>
+__device__ __forceinline__ void write_norm(const float4 (&v)[NV], const LnOut& o, int w_dt, float mean, float var, size_t row, int nvec, int D) {
+    const float rstd = o.w == nullptr ? 1.f : 1.0f / sqrtf(var + o.eps);
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (i >= nvec) continue;
+        const float4 g = o.w == nullptr ? make_float4(1.f, 1.f, 1.f, 1.f) : ld_w4(o.w, w_dt, i);
+        const float4 n = make_float4((v[k].x - mean) * rstd * g.x, (v[k].y - mean) * rstd * g.y, (v[k].z - mean) * rstd * g.z,
+                                     (v[k].w - mean) * rstd * g.w);
+        TO* dst = (TO*)o.out + row * D + 4 * i;
+        if (sizeof(TO) == 4) {
+            *reinterpret_cast<float4*>(dst) = n;
+        } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(n.x, n.y), hi = __floats2bfloat162_rn(n.z, n.w);
+            uint2 pk;
+            pk.x = *reinterpret_cast<uint32_t*>(&lo);
+            pk.y = *reinterpret_cast<uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(dst) = pk;
+        }
+    }
+}
+
+template <typename TO, int NV>
+__global__ void __launch_bounds__(256)
+layernorm_multi_vec_kernel(float* __restrict__ x, LnBranch b0, LnBranch b1, int scale_dt, size_t slice, LnOut o0, LnOut o1, int w_dt,
+                           const int* __restrict__ rows, int D, int rms) {
+    __shared__ float scratch[32];
+    gfb_pdl_launch();
+    gfb_pdl_wait();
+    const int r = blockIdx.x, nvec = D >> 2;
+    const size_t base = (size_t)(rows ? rows[r] : r) * D;
+    float4 v[NV];
+    float4* xr = reinterpret_cast<float4*>(x + base);
+#pragma unroll
+    for (int k = 0; k < NV; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        v[k] = i < nvec ? xr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (b0.y != nullptr) add_branch<NV>(v, b0, scale_dt, slice, base, nvec);
+    if (b1.y != nullptr) add_branch<NV>(v, b1, scale_dt, slice, base, nvec);
+    if (b0.y != nullptr || b1.y != nullptr) {
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < nvec) xr[i] = v[k];
+        }
+    }
+    if (o0.out == nullptr && o1.out == nullptr) return;
+    float mean = 0.f, var = 0.f;
+    if (!(o0.out != nullptr && o0.w == nullptr)) {
+        if (!rms) {
+            float s = 0.f;
+#pragma unroll
+            for (int k = 0; k < NV; k++) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);          // vectors beyond the row are zero
+            mean = gfb_block_sum(s, scratch) / (float)D;
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; k++)
+            if ((int)threadIdx.x + k * (int)blockDim.x < nvec) {
+                const float a = v[k].x - mean, b = v[k].y - mean, c = v[k].z - mean, d = v[k].w - mean;
+                ss += (a * a + b * b) + (c * c + d * d);
+            }
+        var = gfb_block_sum(ss, scratch) / (float)D;
+    }
+    if (o0.out != nullptr) write_norm<TO, NV>(v, o0, w_dt, mean, var, (size_t)r, nvec, D);
+    if (o1.out != nullptr) write_norm<TO, NV>(v, o1, w_dt, mean, var, (size_t)r, nvec, D);
+}
+
 // x float32 [T, D].  Branch b (y_b null: none): float32 [max(S_b,1)][T][D] with the per-column factor scale_b ([D] of
 // scale_dt, or null).  Output k (out_k null: none): [R, D] of out_dt = norm of the new x with weight w_k and eps_k.
-// rows (or null) gathers input rows and cannot be combined with a branch.
+// A null w_k (only w0, and then without a second output): the row itself.  rows (or null) gathers input rows and cannot
+// be combined with a branch.
 GFB_API int gfb_layernorm_multi(float* x, const float* y0, int S0, const void* scale0, const float* y1, int S1,
                                 const void* scale1, int scale_dt, long slice, const void* w0, float eps0, void* out0,
                                 const void* w1, float eps1, void* out1, int w_dt, int out_dt, const int* rows, int R, int D,
@@ -328,8 +443,32 @@ GFB_API int gfb_layernorm_multi(float* x, const float* y0, int S0, const void* s
     if ((y0 != nullptr || y1 != nullptr) && rows != nullptr) return gfb_fail("gfb_layernorm_multi: a branch sum cannot be combined with a row gather");
     if (y0 == nullptr && y1 == nullptr && out0 == nullptr && out1 == nullptr) return 0;
     if ((size_t)D * sizeof(float) > 200 * 1024) return gfb_fail("gfb_layernorm_multi: a row of %d elements does not fit shared memory", D);
+    if ((out1 != nullptr && w1 == nullptr) || (out0 != nullptr && w0 == nullptr && out1 != nullptr))
+        return gfb_fail("gfb_layernorm_multi: the row itself can only be the first and only output");
     LnBranch b0{y0, S0, scale0}, b1{y1, S1, scale1};
     LnOut o0{w0, eps0, out0}, o1{w1, eps1, out1};
+    const bool aligned = (((uintptr_t)x | (uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)scale0 | (uintptr_t)scale1 | (uintptr_t)w0 | (uintptr_t)w1 |
+                           (uintptr_t)out0 | (uintptr_t)out1) & 15) == 0;
+    if (D % 4 == 0 && slice % 4 == 0 && aligned && D <= 4 * LN_VEC * 256) {
+        int per = R <= 256 ? 2 : LN_VEC;                        // as in gfb_layernorm
+        if ((D / 4 + per - 1) / per > 256) per = (D / 4 + 255) / 256;
+        per = per <= 2 ? 2 : per <= 4 ? 4 : LN_VEC;
+        int vthreads = ((D / 4 + per - 1) / per + 31) / 32 * 32;
+        if (vthreads < 64) vthreads = 64;
+        if (vthreads > 256) vthreads = 256;
+        if (D / 4 <= per * vthreads) {
+            cudaError_t ev;
+#define VGO(TO, NV) ev = gfb_launch(layernorm_multi_vec_kernel<TO, NV>, dim3(R), dim3(vthreads), 0, stream, x, b0, b1, scale_dt, \
+                                    (size_t)slice, o0, o1, w_dt, rows, D, rms)
+#define VPICK(TO) do { if (per == 2) VGO(TO, 2); else if (per == 4) VGO(TO, 4); else VGO(TO, 8); } while (0)
+            if ((out0 == nullptr && out1 == nullptr) || out_dt == GFB_F32) VPICK(float);
+            else if (out_dt == GFB_BF16) VPICK(__nv_bfloat16);
+            else return gfb_fail("gfb_layernorm_multi: unknown output type %d", out_dt);
+#undef VPICK
+#undef VGO
+            return gfb_check(ev, "gfb_layernorm_multi (vector)");
+        }
+    }
     const int threads = D >= 2048 ? 512 : (D >= 512 ? 256 : 128);
     const size_t smem = (size_t)D * sizeof(float);
     cudaError_t e;

@@ -3,12 +3,17 @@
 // gfb_moe_router        few tokens: router logits and choice in one launch (a block per token)
 // gfb_moe_route         from 32-bit router logits: s = sigmoid(z); the `top` experts with the largest s + correction
 //                       (lowest index on ties); weights s / (sum of the chosen s + 1e-20) * scale.  Or (mode ROUTE_SOFTMAX_TOP)
-//                       the `top` largest logits themselves, weighted by the softmax over just those, times scale
+//                       the `top` largest logits themselves, weighted by the softmax over just those, times scale.  Or (mode
+//                       ROUTE_SOFTMAX) s = softmax over all E logits, chosen by s + correction, weighted by s * scale.  With
+//                       `groups` > 1 only experts of the `keep` groups (of equal size, neighbours) whose largest choice
+//                       scores are largest can be chosen.  `shared` = 1: every token also runs expert number E with weight 1
 // gfb_moe_glu           act[pair, f] = g * sigmoid(alpha g) * (u + shift),  g = min(gate_f . h, limit),
 //                       u = clamp(up_f . h, -limit, limit), for every (token, chosen expert) pair
-// gfb_moe_down          x[t] += sum over the token's chosen experts of weight * (W_down act[pair]); 32-bit sum into the stream
+//                       or, for experts of two products (kind RELU2), act[pair, f] = max(up_f . h, 0)^2
+// gfb_moe_down          x[t] (+)= sum over the token's chosen experts of weight * (W_down act[pair]); 32-bit sum into the stream
 //
-// The gate and up rows of an expert alternate in one matrix w13 [E, 2F, D], the down matrix is w2 [E, D, F].
+// The gate and up rows of an expert alternate in one matrix w13 [E, 2F, D] (RELU2: the up matrix [E, F, D] alone), the down
+// matrix is w2 [E, D, F].  A shared expert of the experts' own size is one more matrix behind theirs.
 // A pair is p = t * top + r (r: rank of the expert among the token's choices).
 //
 // Two forms of the expert products.  Few tokens (a decode step): a warp per output number streams the weight row once,
@@ -31,21 +36,68 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf
 // ------------------------------------------------------------------------------------ router ----
 constexpr int MAX_EPL = 16;           // experts per lane: E <= 512
 constexpr int ROUTE_WARPS = 4;
-enum { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_TOP = 1 };
+enum { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX = 2 };
+constexpr int MAX_GROUPS = 32;        // a lane keeps a group's score
+
+struct RouteArgs {
+    int E, top;
+    float scale;
+    int mode, groups, keep, shared;
+};
 
 // one token's choice by one warp: `logits` are the token's E router logits
-__device__ __forceinline__ void route_token(const float* __restrict__ logits, const void* __restrict__ correction, int c_dt, int E, int top,
-                                            float scale, int* __restrict__ idx, float* __restrict__ weights, int lane, int mode) {
+__device__ __forceinline__ void route_token(const float* __restrict__ logits, const void* __restrict__ correction, int c_dt,
+                                            const RouteArgs& ra, int* __restrict__ idx, float* __restrict__ weights, int lane) {
+    const int E = ra.E, top = ra.top, mode = ra.mode;
+    const float scale = ra.scale;
     float s[MAX_EPL], c[MAX_EPL];
+    float z_max = -INFINITY, z_inv = 0.f;
+    if (mode == ROUTE_SOFTMAX) {
+        for (int e = lane; e < E; e += 32) z_max = fmaxf(z_max, logits[e]);
+        z_max = gfb_warp_max(z_max);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(logits[e] - z_max);
+        z_inv = 1.0f / gfb_warp_sum(sum);
+    }
 #pragma unroll
     for (int i = 0; i < MAX_EPL; i++) {
         const int e = lane + 32 * i;
         if (e < E) {
-            s[i] = mode == ROUTE_SOFTMAX_TOP ? logits[e] : sigmoid_f(logits[e]);
+            s[i] = mode == ROUTE_SOFTMAX_TOP ? logits[e] : mode == ROUTE_SOFTMAX ? expf(logits[e] - z_max) * z_inv : sigmoid_f(logits[e]);
             c[i] = s[i] + (correction != nullptr ? ldw(correction, c_dt, e) : 0.f);
         } else {
             s[i] = 0.f;
             c[i] = -INFINITY;
+        }
+    }
+    if (ra.groups > 1) {
+        // lane g keeps the largest choice score of group g; the `keep` best groups stay (the lowest index on ties)
+        const int per = E / ra.groups;
+        float score = -INFINITY;
+        for (int g = 0; g < ra.groups; g++) {
+            float m = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < MAX_EPL; i++)
+                if ((lane + 32 * i) / per == g) m = fmaxf(m, c[i]);            // (experts beyond E are -inf)
+            m = gfb_warp_max(m);
+            if (lane == g) score = m;
+        }
+        unsigned kept = 0u;
+        for (int r = 0; r < ra.keep; r++) {
+            float best = (lane < ra.groups && !(kept >> lane & 1u)) ? score : -INFINITY;
+            int best_g = (lane < ra.groups && !(kept >> lane & 1u)) ? lane : 0x7fffffff;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+                if (ob > best || (ob == best && og < best_g)) { best = ob; best_g = og; }
+            }
+            if (best_g < 32) kept |= 1u << best_g;
+        }
+#pragma unroll
+        for (int i = 0; i < MAX_EPL; i++) {
+            const int e = lane + 32 * i;
+            if (e < E && !(kept >> (e / per) & 1u)) c[i] = -INFINITY;
         }
     }
     float sum = 0.f, mine = 0.f;       // lane r keeps the r-th chosen score
@@ -75,28 +127,42 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
     }
     if (lane < top) {
         idx[lane] = mine_e;
-        weights[lane] = mode == ROUTE_SOFTMAX_TOP ? mine / sum * scale : mine / (sum + 1e-20f) * scale;
+        weights[lane] = mode == ROUTE_SOFTMAX ? mine * scale : mode == ROUTE_SOFTMAX_TOP ? mine / sum * scale : mine / (sum + 1e-20f) * scale;
+    }
+    if (ra.shared && lane == 0) {
+        idx[top] = E;
+        weights[top] = 1.f;
     }
 }
 
+static int check_route(const RouteArgs& ra, const char* what) {
+    if (ra.E < 1 || ra.E > 32 * MAX_EPL) return gfb_fail("%s: %d experts (1 to %d)", what, ra.E, 32 * MAX_EPL);
+    if (ra.top < 1 || ra.top > 32 || ra.top > ra.E) return gfb_fail("%s: %d of %d experts per token (1 to 32)", what, ra.top, ra.E);
+    if (ra.groups < 1 || ra.groups > MAX_GROUPS || ra.E % ra.groups || ra.keep < 1 || ra.keep > ra.groups || ra.top > ra.keep * (ra.E / ra.groups))
+        return gfb_fail("%s: %d experts from %d of %d groups of %d experts in all", what, ra.top, ra.keep, ra.groups, ra.E);
+    return 0;
+}
+
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
-moe_route_kernel(const float* __restrict__ logits, int ld, const void* __restrict__ correction, int c_dt, int E, int top,
-                 float scale, int* __restrict__ idx, float* __restrict__ weights, int T, int mode) {
+moe_route_kernel(const float* __restrict__ logits, int ld, const void* __restrict__ correction, int c_dt, RouteArgs ra,
+                 int* __restrict__ idx, float* __restrict__ weights, int T) {
     gfb_pdl_launch();
     gfb_pdl_wait();
     const int lane = threadIdx.x & 31;
     const int t = blockIdx.x * ROUTE_WARPS + (threadIdx.x >> 5);
     if (t >= T) return;
-    route_token(logits + (size_t)t * ld, correction, c_dt, E, top, scale, idx + (size_t)t * top, weights + (size_t)t * top, lane, mode);
+    const size_t at = (size_t)t * (ra.top + ra.shared);
+    route_token(logits + (size_t)t * ld, correction, c_dt, ra, idx + at, weights + at, lane);
 }
 
+// idx int32 and weights float32 [T, top + shared]
 GFB_API int gfb_moe_route(const float* logits, int ld, const void* correction, int c_dt, int E, int top, float scale, int* idx,
-                          float* weights, int T, int mode, cudaStream_t stream) {
+                          float* weights, int T, int mode, int groups, int keep, int shared, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (E < 1 || E > 32 * MAX_EPL) return gfb_fail("gfb_moe_route: %d experts (1 to %d)", E, 32 * MAX_EPL);
-    if (top < 1 || top > 32 || top > E) return gfb_fail("gfb_moe_route: %d of %d experts per token (1 to 32)", top, E);
+    const RouteArgs ra{E, top, scale, mode, groups, keep, shared ? 1 : 0};
+    if (check_route(ra, "gfb_moe_route")) return 1;
     cudaError_t e = gfb_launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(32 * ROUTE_WARPS), 0, stream, logits, ld,
-                               correction, c_dt, E, top, scale, idx, weights, T, mode);
+                               correction, c_dt, ra, idx, weights, T);
     return gfb_check(e, "gfb_moe_route");
 }
 
@@ -134,8 +200,9 @@ constexpr int ROUTER_WARPS = 8;
 
 template <typename T>
 __global__ void __launch_bounds__(32 * ROUTER_WARPS)
-moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, const void* __restrict__ correction, int c_dt, int E, int top,
-                  float scale, int* __restrict__ idx, float* __restrict__ weights, int D, int mode, int n_extra, float* __restrict__ extra) {
+moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, const void* __restrict__ correction, int c_dt, RouteArgs ra,
+                  int* __restrict__ idx, float* __restrict__ weights, int D, int n_extra, float* __restrict__ extra) {
+    const int E = ra.E;
     extern __shared__ __align__(16) float rs[];        // the input [D], then the logits [E + n_extra]
     float* z = rs + D;
     gfb_pdl_launch();
@@ -153,26 +220,28 @@ moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, const v
         }
     }
     __syncthreads();
-    if (warp == 0) route_token(z, correction, c_dt, E, top, scale, idx + (size_t)t * top, weights + (size_t)t * top, lane, mode);
+    const size_t at = (size_t)t * (ra.top + ra.shared);
+    if (warp == 0) route_token(z, correction, c_dt, ra, idx + at, weights + at, lane);
 }
 
 // h [T, D] and router [>= E + n_extra, D] of type dt (further rows are padding); few tokens only: a block per token.
 // The logits of the n_extra rows behind the experts' go to extra float32 [T, n_extra].
 GFB_API int gfb_moe_router(const void* h, const void* router, int dt, const void* correction, int c_dt, int E, int top, float scale,
-                           int* idx, float* weights, int T, int D, int mode, int n_extra, float* extra, cudaStream_t stream) {
+                           int* idx, float* weights, int T, int D, int mode, int groups, int keep, int shared, int n_extra, float* extra,
+                             cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (E < 1 || E > 32 * MAX_EPL) return gfb_fail("gfb_moe_router: %d experts (1 to %d)", E, 32 * MAX_EPL);
-    if (top < 1 || top > 32 || top > E) return gfb_fail("gfb_moe_router: %d of %d experts per token (1 to 32)", top, E);
+    const RouteArgs ra{E, top, scale, mode, groups, keep, shared ? 1 : 0};
+    if (check_route(ra, "gfb_moe_router")) return 1;
     if (n_extra < 0 || (n_extra > 0 && extra == nullptr)) return gfb_fail("gfb_moe_router: %d further rows without a place for their logits", n_extra);
     const size_t smem = (size_t)(D + E + n_extra) * sizeof(float);
     if (smem > 48 * 1024) return gfb_fail("gfb_moe_router: %zu bytes of shared memory", smem);
     cudaError_t e;
     if (dt == GFB_BF16)
         e = gfb_launch(moe_router_kernel<__nv_bfloat16>, dim3((unsigned)T), dim3(32 * ROUTER_WARPS), smem, stream, (const __nv_bfloat16*)h,
-                       (const __nv_bfloat16*)router, correction, c_dt, E, top, scale, idx, weights, D, mode, n_extra, extra);
+                       (const __nv_bfloat16*)router, correction, c_dt, ra, idx, weights, D, n_extra, extra);
     else if (dt == GFB_F32)
         e = gfb_launch(moe_router_kernel<float>, dim3((unsigned)T), dim3(32 * ROUTER_WARPS), smem, stream, (const float*)h, (const float*)router,
-                       correction, c_dt, E, top, scale, idx, weights, D, mode, n_extra, extra);
+                       correction, c_dt, ra, idx, weights, D, n_extra, extra);
     else return gfb_fail("gfb_moe_router: unknown type %d", dt);
     return gfb_check(e, "gfb_moe_router");
 }
@@ -180,7 +249,10 @@ GFB_API int gfb_moe_router(const void* h, const void* router, int dt, const void
 constexpr int GEMV_WARPS = 8;
 constexpr int GLU_PER_WARP = 2;       // hidden units per warp: 4 weight rows in flight
 
-template <typename T>
+enum { KIND_GLU = 0, KIND_RELU2 = 1 };
+__device__ __forceinline__ float relu2_f(float z) { const float p = fmaxf(z, 0.f); return p * p; }
+
+template <typename T, int KIND>
 __global__ void __launch_bounds__(32 * GEMV_WARPS)
 moe_glu_gemv_kernel(const T* __restrict__ h, const int* __restrict__ idx, const T* __restrict__ w13, T* __restrict__ act, int top,
                     int E, int F, int D, float limit, float alpha, float shift) {
@@ -193,24 +265,29 @@ moe_glu_gemv_kernel(const T* __restrict__ h, const int* __restrict__ idx, const 
     for (int i = threadIdx.x; i < D; i += blockDim.x) hs[i] = gfb_to_f32(h[(size_t)t * D + i]);
     __syncthreads();
     if (e < 0 || e >= E) return;
-    const T* w = w13 + (size_t)e * 2 * F * D;
+    const T* w = w13 + (size_t)e * (KIND == KIND_RELU2 ? 1 : 2) * F * D;
     const bool wide = rows_wide(w, D);
     const int f0 = (blockIdx.x * GEMV_WARPS + warp) * GLU_PER_WARP;
 #pragma unroll
     for (int r = 0; r < GLU_PER_WARP; r++) {
         const int f = f0 + r;
         if (f >= F) break;
-        float g = row_dot(w + (size_t)(2 * f) * D, hs, D, lane, wide);
-        float u = row_dot(w + (size_t)(2 * f + 1) * D, hs, D, lane, wide);
-        if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
-        if (lane == 0) act[(size_t)pair * F + f] = gfb_from_f32<T>(g * sigmoid_f(alpha * g) * (u + shift));
+        if constexpr (KIND == KIND_RELU2) {
+            const float u = row_dot(w + (size_t)f * D, hs, D, lane, wide);
+            if (lane == 0) act[(size_t)pair * F + f] = gfb_from_f32<T>(relu2_f(u));
+        } else {
+            float g = row_dot(w + (size_t)(2 * f) * D, hs, D, lane, wide);
+            float u = row_dot(w + (size_t)(2 * f + 1) * D, hs, D, lane, wide);
+            if (limit > 0.f) { g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit); }
+            if (lane == 0) act[(size_t)pair * F + f] = gfb_from_f32<T>(g * sigmoid_f(alpha * g) * (u + shift));
+        }
     }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(32 * GEMV_WARPS)
 moe_down_gemv_kernel(const T* __restrict__ act, const int* __restrict__ idx, const float* __restrict__ weights, const T* __restrict__ w2,
-                     float* __restrict__ x, int top, int E, int F, int D) {
+                     float* __restrict__ x, int top, int E, int F, int D, int store) {
     extern __shared__ __align__(16) float as[];        // [top][F]
     gfb_pdl_launch();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -227,7 +304,7 @@ moe_down_gemv_kernel(const T* __restrict__ act, const int* __restrict__ idx, con
         if (e < 0 || e >= E) continue;
         acc = fmaf(weights[(size_t)t * top + r], row_dot(w2 + ((size_t)e * D + n) * F, as + (size_t)r * F, F, lane, wide), acc);
     }
-    if (lane == 0) x[(size_t)t * D + n] += acc;
+    if (lane == 0) x[(size_t)t * D + n] = store ? acc : x[(size_t)t * D + n] + acc;
 }
 
 template <typename K>
@@ -302,12 +379,14 @@ GFB_API int gfb_moe_plan(const int* idx, int n_pairs, int E, int tile_rows, int*
 }
 
 // Tiles on CUDA cores (the 32-bit path, and bfloat16 shapes the tensor-core tiles do not take): 64 x 64 outputs per block,
-// each one thread's ascending sum over k.  GLU: A = h rows gathered by pair / top, W = w13 of the tile's expert, the
+// each one thread's ascending sum over k.  RELU2: as GLU with W = the up matrix, act[row, n] = max(., 0)^2.  GLU: A = h rows gathered by pair / top, W = w13 of the tile's expert, the
 // output act[row, n / 2] from the gate (even n) and up (odd n) columns.  DOWN: A = act rows (sorted order), W = w2 of
 // the tile's expert, the output y[pair, n] in 32-bit, pair order.
 constexpr int BM = 64, BN = 64, BK = 16;
 
-template <typename T, bool GLU>
+enum { TILES_DOWN = 0, TILES_GLU = 1, TILES_RELU2 = 2 };
+
+template <typename T, int WHAT>
 __global__ void __launch_bounds__(256)
 moe_tiles_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __restrict__ C, const int* __restrict__ row_pair,
                       const int* __restrict__ tile_expert, int top, int N, int K, float limit, float alpha, float shift) {
@@ -322,7 +401,7 @@ moe_tiles_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __
     const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
     if (threadIdx.x < BM) {
         const int p = row_pair[m0 + threadIdx.x];
-        src_row[threadIdx.x] = p < 0 ? -1 : (GLU ? p / top : m0 + (int)threadIdx.x);
+        src_row[threadIdx.x] = p < 0 ? -1 : (WHAT != TILES_DOWN ? p / top : m0 + (int)threadIdx.x);
     }
     __syncthreads();
     const T* We = W + (size_t)e * N * K;
@@ -360,7 +439,14 @@ moe_tiles_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __
         const int r = ty * 4 + i;
         const int p = row_pair[m0 + r];
         if (p < 0) continue;
-        if (GLU) {
+        if (WHAT == TILES_RELU2) {
+            T* out = (T*)C + (size_t)(m0 + r) * N;
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const int n = n0 + tx * 4 + j;
+                if (n < N) out[n] = gfb_from_f32<T>(relu2_f(acc[i][j]));
+            }
+        } else if (WHAT == TILES_GLU) {
             T* out = (T*)C + (size_t)(m0 + r) * (N >> 1);
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
@@ -382,9 +468,9 @@ moe_tiles_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* __
     }
 }
 
-// x[t] += sum_r weights[t, r] * y[t * top + r] in ascending r
+// x[t] += sum_r weights[t, r] * y[t * top + r] in ascending r (store: x[t] = that sum)
 __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __restrict__ weights, float* __restrict__ x, int top,
-                                   int D, long n) {
+                                   int D, long n, int store) {
     gfb_pdl_launch();
     gfb_pdl_wait();
     const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -393,7 +479,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
     const int c = (int)(i - t * D);
     float acc = 0.f;
     for (int r = 0; r < top; r++) acc = fmaf(weights[t * top + r], y[((size_t)t * top + r) * D + c], acc);
-    x[i] += acc;
+    x[i] = store ? acc : x[i] + acc;
 }
 
 // ------------------------------------------------------------------------------------ around the tensor-core tiles ----
@@ -420,10 +506,10 @@ GFB_API int gfb_moe_gather_rows(const void* h, const int* row_pair, void* hs, in
     return gfb_check(e, "gfb_moe_gather_rows");
 }
 
-// x[t] += sum_r weights[t, r] * y[pair_row[t * top + r]] in ascending r; y in the plan's sorted order, D % 4 == 0
+// x[t] += sum_r weights[t, r] * y[pair_row[t * top + r]] in ascending r (store: x[t] = that sum); y in the plan's sorted order, D % 4 == 0
 __global__ void __launch_bounds__(256)
 moe_combine_rows_kernel(const float4* __restrict__ y, const int* __restrict__ pair_row, const float* __restrict__ weights,
-                        float4* __restrict__ x, int top, int vec_per_row, long n) {
+                        float4* __restrict__ x, int top, int vec_per_row, long n, int store) {
     gfb_pdl_launch();
     gfb_pdl_wait();
     const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -438,39 +524,42 @@ moe_combine_rows_kernel(const float4* __restrict__ y, const int* __restrict__ pa
         const float4 v = y[(size_t)row * vec_per_row + c];
         acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
     }
-    float4 o = x[i];
+    float4 o = store ? make_float4(0.f, 0.f, 0.f, 0.f) : x[i];
     o.x += acc.x; o.y += acc.y; o.z += acc.z; o.w += acc.w;
     x[i] = o;
 }
 
 GFB_API int gfb_moe_combine_rows(const float* y, const int* pair_row, const float* weights, float* x, int T, int top, int D,
-                                 cudaStream_t stream) {
+                                 int store, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (D % 4 || ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(x)) & 15))
         return gfb_fail("gfb_moe_combine_rows: rows of %d floats are not whole 16-byte pieces", D);
     const long n = (long)T * (D / 4);
     cudaError_t e = gfb_launch(moe_combine_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const float4*)y, pair_row,
-                               weights, (float4*)x, top, D / 4, n);
+                               weights, (float4*)x, top, D / 4, n, store);
     return gfb_check(e, "gfb_moe_combine_rows");
 }
 
 // h [T, D], w13 [E, 2F, D], act [rows, F] of type dt.  tiles = 0: the few-token form, act in pair order (rows = T * top);
 // otherwise act in the plan's sorted order (rows = max_tiles * 64) and row_pair, tile_expert from gfb_moe_plan with tiles of 64 rows.
-GFB_API int gfb_moe_glu(const void* h, const int* idx, const void* w13, void* act, int dt, int T, int top, int E, int F, int D,
+// kind 1 (RELU2): w13 is the up matrix [E, F, D] and the constants of the gate are not used.
+GFB_API int gfb_moe_glu(const void* h, const int* idx, const void* w13, void* act, int dt, int kind, int T, int top, int E, int F, int D,
                         float limit, float alpha, float shift, const int* row_pair, const int* tile_expert, int max_tiles,
                         cudaStream_t stream) {
     if (T <= 0) return 0;
     typedef __nv_bfloat16 bf16;
     cudaError_t e;
     if (max_tiles > 0) {
-        dim3 grid((2 * F + BN - 1) / BN, max_tiles);
+        const int N = kind == KIND_RELU2 ? F : 2 * F;
+        dim3 grid((N + BN - 1) / BN, max_tiles);
         if (max_tiles > 65535) return gfb_fail("gfb_moe_glu: %d tiles exceed the grid limit", max_tiles);
-        if (dt == GFB_BF16)
-            e = gfb_launch(moe_tiles_simt_kernel<bf16, true>, grid, dim3(256), 0, stream, (const bf16*)h, (const bf16*)w13, act, row_pair,
-                           tile_expert, top, 2 * F, D, limit, alpha, shift);
-        else if (dt == GFB_F32)
-            e = gfb_launch(moe_tiles_simt_kernel<float, true>, grid, dim3(256), 0, stream, (const float*)h, (const float*)w13, act, row_pair,
-                           tile_expert, top, 2 * F, D, limit, alpha, shift);
+#define GO(T, W) e = gfb_launch(moe_tiles_simt_kernel<T, W>, grid, dim3(256), 0, stream, (const T*)h, (const T*)w13, act, row_pair, \
+                                tile_expert, top, N, D, limit, alpha, shift)
+        if (dt == GFB_BF16 && kind == KIND_RELU2) GO(bf16, TILES_RELU2);
+        else if (dt == GFB_BF16) GO(bf16, TILES_GLU);
+        else if (dt == GFB_F32 && kind == KIND_RELU2) GO(float, TILES_RELU2);
+        else if (dt == GFB_F32) GO(float, TILES_GLU);
+#undef GO
         else return gfb_fail("gfb_moe_glu: unknown type %d", dt);
         return gfb_check(e, "gfb_moe_glu (tiles)");
     }
@@ -478,38 +567,41 @@ GFB_API int gfb_moe_glu(const void* h, const int* idx, const void* w13, void* ac
     if (pairs > 65535) return gfb_fail("gfb_moe_glu: %ld pairs exceed the grid limit of the few-token form", pairs);
     const size_t smem = (size_t)D * sizeof(float);
     dim3 grid((F + GEMV_WARPS * GLU_PER_WARP - 1) / (GEMV_WARPS * GLU_PER_WARP), (unsigned)pairs);
-    if (dt == GFB_BF16) {
-        if (allow_smem(moe_glu_gemv_kernel<bf16>, smem, "gfb_moe_glu")) return 1;
-        e = gfb_launch(moe_glu_gemv_kernel<bf16>, grid, dim3(32 * GEMV_WARPS), smem, stream, (const bf16*)h, idx, (const bf16*)w13, (bf16*)act,
-                       top, E, F, D, limit, alpha, shift);
-    } else if (dt == GFB_F32) {
-        if (allow_smem(moe_glu_gemv_kernel<float>, smem, "gfb_moe_glu")) return 1;
-        e = gfb_launch(moe_glu_gemv_kernel<float>, grid, dim3(32 * GEMV_WARPS), smem, stream, (const float*)h, idx, (const float*)w13,
-                       (float*)act, top, E, F, D, limit, alpha, shift);
-    } else return gfb_fail("gfb_moe_glu: unknown type %d", dt);
+#define GO(T, K)                                                                                                                   \
+    do {                                                                                                                          \
+        if (allow_smem(moe_glu_gemv_kernel<T, K>, smem, "gfb_moe_glu")) return 1;                                                 \
+        e = gfb_launch(moe_glu_gemv_kernel<T, K>, grid, dim3(32 * GEMV_WARPS), smem, stream, (const T*)h, idx, (const T*)w13, (T*)act, \
+                       top, E, F, D, limit, alpha, shift);                                                                        \
+    } while (0)
+    if (dt == GFB_BF16 && kind == KIND_RELU2) GO(bf16, KIND_RELU2);
+    else if (dt == GFB_BF16) GO(bf16, KIND_GLU);
+    else if (dt == GFB_F32 && kind == KIND_RELU2) GO(float, KIND_RELU2);
+    else if (dt == GFB_F32) GO(float, KIND_GLU);
+#undef GO
+    else return gfb_fail("gfb_moe_glu: unknown type %d", dt);
     return gfb_check(e, "gfb_moe_glu");
 }
 
 // act as gfb_moe_glu left it; w2 [E, D, F]; x float32 [T, D] += the weighted sum of the chosen experts' outputs.
-// With tiles: y float32 [T * top, D] is scratch for the experts' outputs in pair order.
+// With tiles: y float32 [T * top, D] is scratch for the experts' outputs in pair order.  store: x = the sum instead of +=.
 GFB_API int gfb_moe_down(const void* act, const int* idx, const float* weights, const void* w2, float* x, int dt, int T, int top,
                          int E, int F, int D, const int* row_pair, const int* tile_expert, int max_tiles, float* y,
-                         cudaStream_t stream) {
+                         int store, cudaStream_t stream) {
     if (T <= 0) return 0;
     typedef __nv_bfloat16 bf16;
     cudaError_t e;
     if (max_tiles > 0) {
         dim3 grid((D + BN - 1) / BN, max_tiles);
         if (dt == GFB_BF16)
-            e = gfb_launch(moe_tiles_simt_kernel<bf16, false>, grid, dim3(256), 0, stream, (const bf16*)act, (const bf16*)w2, (void*)y,
+            e = gfb_launch(moe_tiles_simt_kernel<bf16, TILES_DOWN>, grid, dim3(256), 0, stream, (const bf16*)act, (const bf16*)w2, (void*)y,
                            row_pair, tile_expert, top, D, F, 0.f, 0.f, 0.f);
         else if (dt == GFB_F32)
-            e = gfb_launch(moe_tiles_simt_kernel<float, false>, grid, dim3(256), 0, stream, (const float*)act, (const float*)w2, (void*)y,
+            e = gfb_launch(moe_tiles_simt_kernel<float, TILES_DOWN>, grid, dim3(256), 0, stream, (const float*)act, (const float*)w2, (void*)y,
                            row_pair, tile_expert, top, D, F, 0.f, 0.f, 0.f);
         else return gfb_fail("gfb_moe_down: unknown type %d", dt);
         if (gfb_check(e, "gfb_moe_down (tiles)")) return 1;
         const long n = (long)T * D;
-        e = gfb_launch(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const float*)y, weights, x, top, D, n);
+        e = gfb_launch(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (const float*)y, weights, x, top, D, n, store);
         return gfb_check(e, "gfb_moe_down (combine)");
     }
     if (T > 65535) return gfb_fail("gfb_moe_down: %d tokens exceed the grid limit of the few-token form", T);
@@ -518,11 +610,11 @@ GFB_API int gfb_moe_down(const void* act, const int* idx, const float* weights, 
     if (dt == GFB_BF16) {
         if (allow_smem(moe_down_gemv_kernel<bf16>, smem, "gfb_moe_down")) return 1;
         e = gfb_launch(moe_down_gemv_kernel<bf16>, grid, dim3(32 * GEMV_WARPS), smem, stream, (const bf16*)act, idx, weights, (const bf16*)w2,
-                       x, top, E, F, D);
+                       x, top, E, F, D, store);
     } else if (dt == GFB_F32) {
         if (allow_smem(moe_down_gemv_kernel<float>, smem, "gfb_moe_down")) return 1;
         e = gfb_launch(moe_down_gemv_kernel<float>, grid, dim3(32 * GEMV_WARPS), smem, stream, (const float*)act, idx, weights,
-                       (const float*)w2, x, top, E, F, D);
+                       (const float*)w2, x, top, E, F, D, store);
     } else return gfb_fail("gfb_moe_down: unknown type %d", dt);
     return gfb_check(e, "gfb_moe_down");
 }

@@ -16,7 +16,7 @@ from ..cache import Cache, CacheNeeds, EntryView
 from ..config.spec import ModelSpec, PartSpec
 from ..ops.types import BatchMeta
 from ..parts.residual import Residual
-from ..parts import EMBEDDINGS, NORMS, POSITIONS, build_block, build_part
+from ..parts import EMBEDDINGS, JUNCTIONS, NORMS, POSITIONS, build_block, build_part
 from ..weights.loader import ParamSpec
 
 EMBEDDING_CACHE_ENTRY = -1        # the cache entry of the embedding part's per-sequence state (layers count from 0)
@@ -58,8 +58,10 @@ class Transformer:
         self.positions = [obj for _, obj in positions]
         self.final_norm = build_part(NORMS, spec.final_norm, dtype=self.dtype)
         self.embedding = None if spec.embedding is None else build_part(EMBEDDINGS, spec.embedding, dtype=self.dtype)
+        self.junctions = [build_part(JUNCTIONS, ps, dtype=self.dtype) for ps in spec.junctions]
         self.embed_weight = None
         self.head_weight = None
+        self.token_table = None            # [vocab, spec.token_table]: what token inputs read of a token
         self.after_layer = None            # a callable(Residual) run behind every layer of a step (tests look at the stream)
 
     # ---- parameters -------------------------------------------------------------
@@ -71,6 +73,11 @@ class Transformer:
         if self.embedding is not None:
             for name, s in self.embedding.param_specs().items():
                 specs[f"embedding.{name}"] = s
+        if self.spec.token_table:
+            specs["token_table.weight"] = ParamSpec((self.vocab_size, self.spec.token_table))
+        for i, j in enumerate(self.junctions):
+            for name, s in j.param_specs().items():
+                specs[f"junctions.{i}.{name}"] = s
         for i, b in enumerate(self.blocks):
             for pname, part in b.parts().items():
                 for name, s in part.param_specs().items():
@@ -96,9 +103,14 @@ class Transformer:
         self.final_norm.load(sub("final_norm."))
         if self.embedding is not None:
             self.embedding.load(sub("embedding."))
+        for i, j in enumerate(self.junctions):
+            j.load(sub(f"junctions.{i}."))
+        self.token_table = tensors.get("token_table.weight")
         for i, b in enumerate(self.blocks):
             for pname, part in b.parts().items():
                 part.load(sub(f"layers.{i}.{pname}."))
+                if hasattr(part, "bind_token_table"):
+                    part.bind_token_table(self.token_table)
 
     def export_params(self) -> Dict[str, torch.Tensor]:
         """Every parameter under the name and in the layout of `param_specs` (the inverse of `load_params`);
@@ -109,6 +121,11 @@ class Transformer:
         if self.embedding is not None:
             for name, t in self.embedding.export().items():
                 out[f"embedding.{name}"] = t
+        if self.token_table is not None:
+            out["token_table.weight"] = self.token_table
+        for i, j in enumerate(self.junctions):
+            for name, t in j.export().items():
+                out[f"junctions.{i}.{name}"] = t
         for i, b in enumerate(self.blocks):
             for pname, part in b.parts().items():
                 if not hasattr(part, "export"):
@@ -120,7 +137,7 @@ class Transformer:
     def graph_safe(self) -> bool:
         """Whether a step of this model may be captured in a CUDA graph: every part launches kernels only.  A part
         that reads device values on the host says so with `graph_safe = False`."""
-        parts = [self.final_norm] + [p for b in self.blocks for p in b.parts().values()] + list(self.positions)
+        parts = [self.final_norm] + [p for b in self.blocks for p in b.parts().values()] + list(self.positions) + self.junctions
         if self.embedding is not None:
             parts.append(self.embedding)
         return all(getattr(p, "graph_safe", True) for p in parts + list(self.blocks))
@@ -135,6 +152,8 @@ class Transformer:
                 seen.add(t.data_ptr())
                 total += t.numel() * t.element_size()
         add(self.head_weight)
+        if self.token_table is not None:
+            seen.add(self.token_table.data_ptr())          # a row per token, not the table
         if with_embedding:
             add(self.embed_weight)
         for e in self.spec.schedule:
@@ -142,6 +161,10 @@ class Transformer:
                 for v in vars(part).values():
                     if isinstance(v, torch.Tensor):
                         add(v)
+        for part in self.junctions:
+            for v in vars(part).values():
+                if isinstance(v, torch.Tensor):
+                    add(v)
         for v in vars(self.final_norm).values():
             if isinstance(v, torch.Tensor):
                 add(v)
@@ -192,14 +215,20 @@ class Transformer:
         and values to the cache; the caller advances the lengths afterwards."""
         T = batch.n_tokens
         ops.set_launch_overlap(self.spec.launch_overlap)
+        batch.tokens = tokens
         x = torch.empty(T, self.dim, dtype=torch.float32, device=self.device)
         scale = 1.0 if self.spec.embed_scale is None else float(self.spec.embed_scale)
         if self.embedding is None:
             ops.embed(tokens, self.embed_weight, x, batch.status, scale)
         else:
             self.embedding.forward(tokens, self.embed_weight, x, batch, cache.view(EMBEDDING_CACHE_ENTRY), scale)
+        x0 = x                                  # the embedding output, which junctions read again
+        if self.junctions and self.spec.schedule[0].junction is None:
+            x = x0.clone()                      # layers ahead of the first junction write into the stream
         x = Residual(x)
         for e in self.spec.schedule:
+            if e.junction is not None:
+                self.junctions[e.junction].forward(x, x0, e.turn)
             if e.kv_from is None:
                 self.blocks[e.layer].forward(x, batch, cache.view(e.cache), append=e.owns_cache)
             else:

@@ -141,7 +141,7 @@ def layernorm_multi(x, branches=(), outs=(), rows=None, rms: bool = False):
     """One row, one mean and variance, several norms.  x float32 [T, D].  branches: up to two (y, scale): first
     x += scale * y (written back), y a float32 [T, D] tensor or partial sums [S, T, D] added in ascending order,
     scale a per-column factor [D] or None.  outs: up to two (weight, eps, out): out [R, D] = (x - mean) / sqrt(var +
-    eps) * weight in the compute type.  rows int32 [R] gathers input rows (not together with branches).  rms=True:
+    eps) * weight in the compute type; weight None (one output only): the new row itself.  rows int32 [R] gathers input rows (not together with branches).  rms=True:
     the root-mean-square form (no mean)."""
     return kernels().layernorm_multi(x, branches, outs, rows, rms)
 
@@ -159,11 +159,37 @@ def latent_prepare(src, q_off: int, kv_off: int, q_out, kv: PagedKV, batch: Batc
 
 
 def headwise_linear(a, w, out, n_head: int, k: int, n: int, a_off: int = 0, a_stride: Optional[int] = None, out_off: int = 0,
-                    out_stride: Optional[int] = None, gate=None, gate_off: int = 0):
+                    out_stride: Optional[int] = None, gate=None, gate_off: int = 0, gate_per_head: bool = False):
     """A product with a weight per head: out[t, h, :] = a[t, h, :] W_h.  a [T, Wa]: head h's k inputs start at column
     a_off + h * a_stride; out [T, Wo]: its n outputs at out_off + h * out_stride; w [n_head, k, n].  gate [T, Wg] (or
-    None): the result is multiplied by sigmoid(gate[t, gate_off + h * n + j])."""
+    None): the result is multiplied by sigmoid(gate[t, gate_off + h * n + j]), with gate_per_head by
+    sigmoid(gate[t, gate_off + h])."""
+    if gate_per_head:
+        return kernels().headwise_linear(a, w, out, n_head, k, n, a_off, a_stride, out_off, out_stride, gate, gate_off, gate_per_head=True)
     return kernels().headwise_linear(a, w, out, n_head, k, n, a_off, a_stride, out_off, out_stride, gate, gate_off)
+
+
+def gla(src, offsets, rank: int, a2, bias, tau: float, state, state_off: int, norm, eps: float, out, batch: BatchMeta, n_head: int,
+        head_dim: int, v_head_dim: int, q_scale: float):
+    """Gated linear attention over the tokens of a step: with q, k (n_head heads of head_dim), v (n_head heads of v_head_dim),
+    `rank` low-rank numbers and the gate (n_head * v_head_dim) at the column offsets `offsets` = (q, k, v, low, gate) of
+    src [T, W], and z = low a2^T + bias (a2 [n_head * head_dim, rank]), token after token and per head
+    S <- diag(sigmoid(z)^(1/tau)) S + k v^T;  o = S^T (q_scale q);
+    out[t, h, :] = o / sqrt(mean(o^2) + eps) * norm * silu(gate).
+    state float32 [n_slots, S] holds [n_head, head_dim, v_head_dim] per sequence from column state_off; norm [v_head_dim];
+    out [T, n_head * v_head_dim] of src's type.  Decays, state and norm are 32-bit."""
+    return kernels().gla(src, offsets, rank, a2, bias, tau, state, state_off, norm, eps, out, batch, n_head, head_dim, v_head_dim, q_scale)
+
+
+def token_gate(z, tokens, table, off: int, out, status):
+    """out[t, j] = gelu_tanh(z[t, j]) * table[tokens[t], off + j].  z float32 [T, n]; table [V, W]; out [T, n] of the table's
+    type."""
+    return kernels().token_gate(z, tokens, table, off, out, status)
+
+
+def pass_entry(x, x0, step, cat, y):
+    """cat [T, 2 D] = [x ; x0] in the compute type and y [T, D] = step in every row.  x, x0, y float32; step [D]."""
+    return kernels().pass_entry(x, x0, step, cat, y)
 
 
 def short_conv(src, col_off: int, channels: int, weight, bias, state, state_off: int, out, batch: BatchMeta, act: bool = True,
@@ -286,17 +312,29 @@ def sigmoid_gate(y, gate, gate_off: int, group: int):
     return kernels().sigmoid_gate(y, gate, gate_off, group)
 
 
-def moe_route(logits, correction, top: int, scale: float, idx, weights, score: str = "sigmoid"):
+def moe_route(logits, correction, top: int, scale: float, idx, weights, score: str = "sigmoid", groups=None, shared: bool = False):
     """Choice of experts.  logits float32 [T, >= E] (the first E columns count, E = len(correction)): s = sigmoid(logits);
     the `top` experts with the largest s + correction (lowest index on ties) go to idx int32 [T, top], and
     weights float32 [T, top] = their s / (sum of the chosen s + 1e-20) * scale.  score 'softmax_top': the `top` largest
-    logits (+ correction) are chosen and weights = softmax over the chosen logits * scale."""
-    if score == "sigmoid":
-        return kernels().moe_route(logits, correction, top, scale, idx, weights)
-    return kernels().moe_route(logits, correction, top, scale, idx, weights, score=score)
+    logits (+ correction) are chosen and weights = softmax over the chosen logits * scale.  score 'softmax': s = softmax over
+    all E logits, weights = the chosen s * scale.  groups = (count, keep): the experts are `count` equal groups of neighbours
+    and only those of the `keep` groups with the largest single choice score can be chosen.  shared: idx and weights are
+    [T, top + 1] and the last entry of every row is expert number E with weight 1."""
+    kw = _route_options(score, groups, shared)
+    return kernels().moe_route(logits, correction, top, scale, idx, weights, **kw)
 
 
-def moe_router(h, router, correction, top: int, scale: float, idx, weights, score: str = "sigmoid", n_extra: int = 0):
+def _route_options(score, groups, shared) -> dict:
+    kw = {} if score == "sigmoid" else {"score": score}
+    if groups is not None and tuple(groups)[0] > 1:
+        kw["groups"] = (int(groups[0]), int(groups[1]))
+    if shared:
+        kw["shared"] = True
+    return kw
+
+
+def moe_router(h, router, correction, top: int, scale: float, idx, weights, score: str = "sigmoid", n_extra: int = 0, groups=None,
+               shared: bool = False):
     """Router logits z = h router^T (32-bit) and `moe_route` on them.  h [T, D]; router [>= E + n_extra, D] (rows beyond
     those are padding).  A set of kernels may do both in one launch (`moe_router` returning True); otherwise the
     product and the choice run one after the other.  n_extra: that many rows behind the experts' are further 32-bit
@@ -305,25 +343,32 @@ def moe_router(h, router, correction, top: int, scale: float, idx, weights, scor
     k = kernels()
     fused = getattr(k, "moe_router", None)
     E = correction.shape[0]
+    kw = _route_options(score, groups, shared)
     if fused is not None:
-        if score == "sigmoid" and n_extra == 0:
-            if fused(h, router, correction, top, scale, idx, weights):
-                return None
-        else:
-            extra = torch.empty(h.shape[0], n_extra, dtype=torch.float32, device=h.device) if n_extra else None
-            if fused(h, router, correction, top, scale, idx, weights, score=score, extra=extra):
-                return None if extra is None else (extra, 0)
+        extra = None
+        if n_extra:
+            extra = torch.empty(h.shape[0], n_extra, dtype=torch.float32, device=h.device)
+            kw["extra"] = extra
+        if fused(h, router, correction, top, scale, idx, weights, **kw):
+            return None if extra is None else (extra, 0)
+        kw.pop("extra", None)
     z = torch.empty(h.shape[0], router.shape[0], dtype=torch.float32, device=h.device)
     linear(h, router, z)
-    moe_route(z, correction, top, scale, idx, weights, score)
+    k.moe_route(z, correction, top, scale, idx, weights, **kw)
     return (z, E) if n_extra else None
 
 
-def moe_experts(h, idx, weights, w13, w2, x, limit: float, alpha: float, shift: float = 1.0):
+def moe_experts(h, idx, weights, w13, w2, x, limit: float, alpha: float, shift: float = 1.0, act: str = "glu", store: bool = False):
     """x float32 [T, D] += sum_r weights[t, r] * W2_e (g * sigmoid(alpha g) * (u + shift)), e = idx[t, r],
     g = min(gate_e h, limit), u = clamp(up_e h, -limit, limit) (limit <= 0: no clamps).  w13 [E, 2F, D]: rows alternate
-    gate, up; w2 [E, D, F]; h [T, D] of the weights' type."""
-    return kernels().moe_experts(h, idx, weights, w13, w2, x, limit, alpha, shift)
+    gate, up; w2 [E, D, F]; h [T, D] of the weights' type.  act 'relu2': experts of two products, W2_e max(up_e h, 0)^2 with
+    w13 = the up matrices [E, F, D].  store: x = the sum (what it held is not read)."""
+    kw = {}
+    if act != "glu":
+        kw["act"] = act
+    if store:
+        kw["store"] = True
+    return kernels().moe_experts(h, idx, weights, w13, w2, x, limit, alpha, shift, **kw)
 
 
 def activation(x, kind: str, out=None):

@@ -291,9 +291,13 @@ class CudaKernels:
         for w, eps, out in list(outs) + [(None, 0.0, None)] * (2 - len(outs)):
             if out is not None:
                 R = out.shape[0]
-                _need(w, shape=(D,), name="norm weight")
+                if w is not None:
+                    _need(w, shape=(D,), name="norm weight")
+                    w_dt = _dt(w)
+                elif len(outs) > 1:
+                    _fail("the row itself can only be the one output")
                 _need(out, shape=(R, D), name="norm output")
-                w_dt, out_dt = _dt(w), _dt(out)
+                out_dt = _dt(out)
             o_args += [_ptr(w), c_float(eps), _ptr(out)]
         if len(outs) == 2 and (outs[0][0].dtype != outs[1][0].dtype or outs[0][2].dtype != outs[1][2].dtype
                                or outs[0][2].shape != outs[1][2].shape):
@@ -330,7 +334,8 @@ class CudaKernels:
                    c_float(eps), c_int(n_head), c_int(head_dim), c_int(rot_dim), c_int(rank), c_int(_PAIRING[pairing]),
                    c_int(1 if append else 0), _ptr(batch.status), _stream())
 
-    def headwise_linear(self, a, w, out, n_head, k, n, a_off=0, a_stride=None, out_off=0, out_stride=None, gate=None, gate_off=0):
+    def headwise_linear(self, a, w, out, n_head, k, n, a_off=0, a_stride=None, out_off=0, out_stride=None, gate=None, gate_off=0,
+                        gate_per_head=False):
         T = a.shape[0]
         a_stride = k if a_stride is None else a_stride
         out_stride = n if out_stride is None else out_stride
@@ -343,10 +348,11 @@ class CudaKernels:
             _fail("head-wise product: the heads do not fit the rows")
         if gate is not None:
             _need(gate, a.dtype, name="gate")
-            if gate.shape[0] != T or gate_off + n_head * n > gate.shape[1]:
+            if gate.shape[0] != T or gate_off + n_head * (1 if gate_per_head else n) > gate.shape[1]:
                 _fail("head-wise product: the gate does not fit")
         self._call("latent", "gfb_headwise_linear", _ptr(a), c_int(_dt(a)), c_int(a.shape[1]), c_int(a_off), c_int(a_stride), _ptr(w), _ptr(out), c_int(out.shape[1]), c_int(out_off), c_int(out_stride), _ptr(gate),
-                   c_int(gate.shape[1] if gate is not None else 0), c_int(gate_off), c_int(T), c_int(n_head), c_int(k), c_int(n),
+                   c_int(gate.shape[1] if gate is not None else 0), c_int(gate_off), c_int(1 if gate_per_head else n), c_int(T), c_int(n_head),
+                   c_int(k), c_int(n),
                    _stream())
 
     @staticmethod
@@ -355,6 +361,60 @@ class CudaKernels:
         if state.dim() != 2 or state_off < 0 or state_off + need > state.shape[1]:
             _fail(f"{need} numbers of state at column {state_off} do not fit rows of {tuple(state.shape)}")
         return c_void_p(state.data_ptr() + 4 * state_off), c_long(state.shape[1])
+
+    _LOG2E = 1.4426950408889634
+
+    def gla(self, src, offsets, rank, a2, bias, tau, state, state_off, norm, eps, out, batch, n_head, head_dim, v_head_dim, q_scale):
+        T = batch.n_tokens
+        H, d, dv = n_head, head_dim, v_head_dim
+        W = src.shape[1]
+        q_off, k_off, v_off, low_off, g_off = offsets
+        _need(src, shape=(T, W), name="projection")
+        if max(q_off + H * d, k_off + H * d, v_off + H * dv, low_off + rank, g_off + H * dv) > W:
+            _fail(f"q, k, v, low-rank inputs and gate at {offsets} do not fit rows of {W}")
+        _need(a2, src.dtype, (H * d, rank), "decay weights")
+        _need(bias, shape=(H * d,), name="decay bias")
+        _need(norm, shape=(dv,), name="head norm weight")
+        _need(out, src.dtype, (T, H * dv), "gated output")
+        if not tau > 0:
+            _fail(f"tau = {tau} must be positive")
+        sp, sld = self._state_args(state, state_off, H * d * dv)
+        factor = c_float(self._LOG2E / tau)
+        cols = (c_int(q_off), c_int(k_off), c_int(v_off), c_int(low_off))
+        if (batch.max_q_len == 1 and T == batch.n_seqs and dv % 4 == 0 and dv <= 2048 and state.shape[1] % 4 == 0 and sp.value % 16 == 0
+                and (512 // (dv // 4) * dv + 3 * d + rank) * 4 <= 48 * 1024):
+            return self._call("gla", "gfb_gla_decode", _ptr(src), c_int(_dt(src)), c_int(W), *cols, c_int(g_off), c_int(rank), _ptr(a2),
+                              _ptr(bias), c_int(_dt(bias)), factor, sp, sld, _ptr(norm), c_int(_dt(norm)), c_float(eps), _ptr(out),
+                              *self._batch_args(batch), c_int(H), c_int(d), c_int(dv), c_float(q_scale), _stream())
+        fn = self._f("gla", "gfb_gla_scratch_floats")
+        fn.restype = c_long
+        scratch = torch.empty(fn(c_int(T), c_int(batch.n_seqs), c_int(H), c_int(d), c_int(dv)), dtype=torch.float32, device=src.device)
+        o = torch.empty(T, H * dv, dtype=torch.float32, device=src.device)
+        self._call("gla", "gfb_gla", _ptr(src), c_int(_dt(src)), c_int(W), *cols, c_int(rank), _ptr(a2), _ptr(bias), c_int(_dt(bias)), factor,
+                   sp, sld, _ptr(o), _ptr(scratch), *self._batch_args(batch), c_int(H), c_int(d), c_int(dv), c_float(q_scale), _stream())
+        self.gated_norm(o, src, g_off, norm, out, dv, eps, act="silu", gate_first=False)
+
+    def token_gate(self, z, tokens, table, off, out, status):
+        T, n = z.shape
+        V, W = table.shape
+        _need(z, torch.float32, name="gate input")
+        _need(tokens, torch.int32, (T,), "tokens")
+        _need(table, name="side table")
+        _need(out, table.dtype, (T, n), "gated side rows")
+        if off < 0 or off + n > W:
+            _fail(f"columns {off} .. {off + n - 1} of a side table of {W}")
+        self._call("embedding", "gfb_token_gate", _ptr(tokens), _ptr(table), c_int(_dt(table)), c_int(V), c_int(W), c_int(off), _ptr(z), _ptr(out),
+                   c_int(_dt(out)), c_int(T), c_int(n), _ptr(status), _stream())
+
+    def pass_entry(self, x, x0, step, cat, y):
+        T, D = x.shape
+        _need(x, torch.float32, name="stream")
+        _need(x0, torch.float32, (T, D), "embedding output")
+        _need(step, shape=(D,), name="vector of the pass")
+        _need(cat, shape=(T, 2 * D), name="input of the entry product")
+        _need(y, torch.float32, (T, D), "new stream")
+        self._call("elementwise", "gfb_pass_entry", _ptr(x), _ptr(x0), _ptr(step), c_int(_dt(step)), _ptr(cat), c_int(_dt(cat)), _ptr(y), c_int(T),
+                   c_int(D), _stream())
 
     def short_conv(self, src, col_off, channels, weight, bias, state, state_off, out, batch, act=True, in_bias=None):
         T = batch.n_tokens
@@ -551,10 +611,16 @@ class CudaKernels:
     MOE_PAIR_ROWS_PER_EXPERT = 384     # (token, expert) pairs per expert from which the row tiles have 256 rows
     _EPI_GLU_CLAMP = 8
 
-    _ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1}
+    _ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1, "softmax": 2}
+    MOE_MAX_GROUPS = 32
 
-    def moe_route(self, logits, correction, top, scale, idx, weights, score="sigmoid"):
-        T = logits.shape[0]
+    def _route_args(self, score, groups, shared):
+        if score not in self._ROUTE_SCORES:
+            _fail(f"unknown router score '{score}'")
+        return (c_int(self._ROUTE_SCORES[score]), c_int(groups[0]), c_int(groups[1]), c_int(1 if shared else 0))
+
+    def moe_route(self, logits, correction, top, scale, idx, weights, score="sigmoid", groups=(1, 1), shared=False):
+        T, slots = logits.shape[0], top + (1 if shared else 0)
         if score not in self._ROUTE_SCORES:
             _fail(f"unknown router score '{score}'")
         E = correction.shape[0]
@@ -562,15 +628,17 @@ class CudaKernels:
         if logits.dim() != 2 or logits.shape[1] < E:
             _fail(f"router logits {tuple(logits.shape)} for {E} experts")
         _need(correction, name="router correction")
-        _need(idx, torch.int32, (T, top), "chosen experts")
-        _need(weights, torch.float32, (T, top), "expert weights")
+        _need(idx, torch.int32, (T, slots), "chosen experts")
+        _need(weights, torch.float32, (T, slots), "expert weights")
         self._call("moe", "gfb_moe_route", _ptr(logits), c_int(logits.shape[1]), _ptr(correction), c_int(_dt(correction)), c_int(E),
-                   c_int(top), c_float(scale), _ptr(idx), _ptr(weights), c_int(T), c_int(self._ROUTE_SCORES[score]), _stream())
+                   c_int(top), c_float(scale), _ptr(idx), _ptr(weights), c_int(T), *self._route_args(score, groups, shared), _stream())
 
     MOE_ROUTER_FEW_TOKENS = 64         # up to this many tokens the router's product and its choice are one launch
 
-    def moe_router(self, h, router, correction, top, scale, idx, weights, score="sigmoid", extra=None) -> bool:
+    def moe_router(self, h, router, correction, top, scale, idx, weights, score="sigmoid", extra=None, groups=(1, 1),
+                   shared=False) -> bool:
         T, D = h.shape
+        slots = top + (1 if shared else 0)
         E = correction.shape[0]
         n_extra = 0 if extra is None else extra.shape[1]
         if T > self.MOE_ROUTER_FEW_TOKENS or (D + E + n_extra) * 4 > 48 * 1024:
@@ -584,26 +652,30 @@ class CudaKernels:
         if router.shape[0] < E + n_extra:
             _fail(f"router weights {tuple(router.shape)} for {E} experts and {n_extra} further rows")
         _need(correction, name="router correction")
-        _need(idx, torch.int32, (T, top), "chosen experts")
-        _need(weights, torch.float32, (T, top), "expert weights")
+        _need(idx, torch.int32, (T, slots), "chosen experts")
+        _need(weights, torch.float32, (T, slots), "expert weights")
         self._call("moe", "gfb_moe_router", _ptr(h), _ptr(router), c_int(_dt(h)), _ptr(correction), c_int(_dt(correction)), c_int(E),
-                   c_int(top), c_float(scale), _ptr(idx), _ptr(weights), c_int(T), c_int(D), c_int(self._ROUTE_SCORES[score]),
+                   c_int(top), c_float(scale), _ptr(idx), _ptr(weights), c_int(T), c_int(D), *self._route_args(score, groups, shared),
                    c_int(n_extra), _ptr(extra), _stream())
         return True
 
-    def moe_experts(self, h, idx, weights, w13, w2, x, limit, alpha, shift=1.0):
+    def moe_experts(self, h, idx, weights, w13, w2, x, limit, alpha, shift=1.0, act="glu", store=False):
         T, D = h.shape
-        E, F2, _ = w13.shape
-        F, top = F2 // 2, idx.shape[1]
+        E, N1, _ = w13.shape                            # rows of an expert's first matrix
+        if act not in ("glu", "relu2"):
+            _fail(f"unknown activation of the experts '{act}'")
+        relu2 = act == "relu2"
+        F, top = N1 if relu2 else N1 // 2, idx.shape[1]
+        kind, keep = c_int(1 if relu2 else 0), c_int(1 if store else 0)
         _need(h, name="expert input")
-        _need(w13, h.dtype, (E, 2 * F, D), "gate/up weights")
+        _need(w13, h.dtype, (E, N1, D), "gate/up weights")
         _need(w2, h.dtype, (E, D, F), "down weights")
         _need(idx, torch.int32, (T, top), "chosen experts")
         _need(weights, torch.float32, (T, top), "expert weights")
         _need(x, torch.float32, (T, D), "residual stream")
         dt = c_int(_dt(h))
         sizes = (c_int(T), c_int(top), c_int(E), c_int(F), c_int(D))
-        if h.dtype == torch.bfloat16 and T > self.MOE_TC_FEW_TOKENS and D % 8 == 0 and F % 8 == 0 and E * max(2 * F, D) < 2 ** 31:
+        if h.dtype == torch.bfloat16 and T > self.MOE_TC_FEW_TOKENS and D % 8 == 0 and F % 8 == 0 and E * max(N1, D) < 2 ** 31:
             # sorted by expert in tiles of 128 rows, both products on the tensor cores: gather the rows, gate/up with the
             # activation in the epilogue, down into 32-bit rows, then the weighted sum into the stream in pair order
             pairs = T * top
@@ -620,25 +692,25 @@ class CudaKernels:
                        _ptr(tile_expert), c_int(tiles), _ptr(tiles_used), _stream())
             hs = torch.empty(tiles * rows, D, dtype=h.dtype, device=h.device)
             self._call("moe", "gfb_moe_gather_rows", _ptr(h), _ptr(row_pair), _ptr(hs), c_int(tiles * rows), c_int(top), c_int(D), _stream())
-            act = torch.empty(tiles * rows, F, dtype=h.dtype, device=h.device)
-            self._label = f"moe_glu_tc {2 * F}x{D}"
-            self._call("gemm_tc", "gfb_gemm_tc_grouped", _ptr(hs), _ptr(w13), _ptr(act), c_int(_dt(act)), c_int(tiles * rows), c_int(rows), c_int(E),
-                       c_int(2 * F), c_int(D), c_int(self._EPI_GLU_CLAMP), _ptr(tile_expert), _ptr(tiles_used), c_float(limit), c_float(alpha),
+            mid = torch.empty(tiles * rows, F, dtype=h.dtype, device=h.device)
+            self._label = f"moe_{act}_tc {N1}x{D}"
+            self._call("gemm_tc", "gfb_gemm_tc_grouped", _ptr(hs), _ptr(w13), _ptr(mid), c_int(_dt(mid)), c_int(tiles * rows), c_int(rows), c_int(E),
+                       c_int(N1), c_int(D), c_int(_EPI["relu2"] if relu2 else self._EPI_GLU_CLAMP), _ptr(tile_expert), _ptr(tiles_used), c_float(limit), c_float(alpha),
                        c_float(shift), _ptr(self.status), _stream())
             y = torch.empty(tiles * rows, D, dtype=torch.float32, device=h.device)
             self._label = f"moe_down_tc {D}x{F}"
-            self._call("gemm_tc", "gfb_gemm_tc_grouped", _ptr(act), _ptr(w2), _ptr(y), c_int(_dt(y)), c_int(tiles * rows), c_int(rows), c_int(E),
+            self._call("gemm_tc", "gfb_gemm_tc_grouped", _ptr(mid), _ptr(w2), _ptr(y), c_int(_dt(y)), c_int(tiles * rows), c_int(rows), c_int(E),
                        c_int(D), c_int(F), c_int(_EPI["store"]), _ptr(tile_expert), _ptr(tiles_used), c_float(0.0), c_float(0.0), c_float(0.0),
                        _ptr(self.status), _stream())
-            self._call("moe", "gfb_moe_combine_rows", _ptr(y), _ptr(pair_row), _ptr(weights), _ptr(x), c_int(T), c_int(top), c_int(D),
+            self._call("moe", "gfb_moe_combine_rows", _ptr(y), _ptr(pair_row), _ptr(weights), _ptr(x), c_int(T), c_int(top), c_int(D), keep,
                        _stream())
             return
         if T <= self.MOE_FEW_TOKENS:
-            act = torch.empty(T * top, F, dtype=h.dtype, device=h.device)
-            self._call("moe", "gfb_moe_glu", _ptr(h), _ptr(idx), _ptr(w13), _ptr(act), dt, *sizes, c_float(limit), c_float(alpha),
+            mid = torch.empty(T * top, F, dtype=h.dtype, device=h.device)
+            self._call("moe", "gfb_moe_glu", _ptr(h), _ptr(idx), _ptr(w13), _ptr(mid), dt, kind, *sizes, c_float(limit), c_float(alpha),
                        c_float(shift), _ptr(None), _ptr(None), c_int(0), _stream())
-            self._call("moe", "gfb_moe_down", _ptr(act), _ptr(idx), _ptr(weights), _ptr(w2), _ptr(x), dt, *sizes, _ptr(None), _ptr(None),
-                       c_int(0), _ptr(None), _stream())
+            self._call("moe", "gfb_moe_down", _ptr(mid), _ptr(idx), _ptr(weights), _ptr(w2), _ptr(x), dt, *sizes, _ptr(None), _ptr(None),
+                       c_int(0), _ptr(None), keep, _stream())
             return
         # the sorted form: pairs grouped by expert, every expert's rows padded to whole tiles
         rows = self.MOE_TILE_ROWS
@@ -648,12 +720,12 @@ class CudaKernels:
         row_pair, pair_row, tile_expert = plan[:tiles * rows], plan[tiles * rows:tiles * rows + pairs], plan[tiles * rows + pairs:]
         self._call("moe", "gfb_moe_plan", _ptr(idx), c_int(pairs), c_int(E), c_int(rows), _ptr(row_pair), _ptr(pair_row),
                    _ptr(tile_expert), c_int(tiles), _ptr(None), _stream())
-        act = torch.empty(tiles * rows, F, dtype=h.dtype, device=h.device)
+        mid = torch.empty(tiles * rows, F, dtype=h.dtype, device=h.device)
         y = torch.empty(pairs, D, dtype=torch.float32, device=h.device)
-        self._call("moe", "gfb_moe_glu", _ptr(h), _ptr(idx), _ptr(w13), _ptr(act), dt, *sizes, c_float(limit), c_float(alpha),
+        self._call("moe", "gfb_moe_glu", _ptr(h), _ptr(idx), _ptr(w13), _ptr(mid), dt, kind, *sizes, c_float(limit), c_float(alpha),
                    c_float(shift), _ptr(row_pair), _ptr(tile_expert), c_int(tiles), _stream())
-        self._call("moe", "gfb_moe_down", _ptr(act), _ptr(idx), _ptr(weights), _ptr(w2), _ptr(x), dt, *sizes, _ptr(row_pair),
-                   _ptr(tile_expert), c_int(tiles), _ptr(y), _stream())
+        self._call("moe", "gfb_moe_down", _ptr(mid), _ptr(idx), _ptr(weights), _ptr(w2), _ptr(x), dt, *sizes, _ptr(row_pair),
+                   _ptr(tile_expert), c_int(tiles), _ptr(y), keep, _stream())
 
     def activation(self, x, kind, out=None):
         if kind not in _UNARY:
@@ -787,23 +859,24 @@ class CudaKernels:
         capped = bool(softcap) or bool(keep_first)                    # the tensor-core kernels have these at head sizes 64 and 128
         special = capped or maps != 1
         plain = chunk is None and sink is None and not biased and not special
-        if (values_in_keys and not biased and not special and q.dtype == torch.bfloat16 and n_kv == 1 and chunk is None and sink is None
-                and not window and head_dim % 16 == 0 and dv % 16 == 0 and dv <= 512 and dv < head_dim and kv.page_size % 32 == 0
+        if (values_in_keys and not biased and not special and q.dtype == torch.bfloat16 and n_kv == 1 and chunk is None
+                and head_dim % 16 == 0 and dv % 16 == 0 and dv <= 512 and dv < head_dim and kv.page_size % 32 == 0
                 and (64 + 2 * 32) * (head_dim + 8) * 2 <= 220 * 1024):
             # a latent that all heads share: the tensor-core kernel that fetches every cached row once per 64 (token, head)
             # pairs of a sequence (a decode step's heads are the rows of one MMA)
             splits, scratch = 1, None
             if batch.max_q_len == 1:
                 # a decode step: slices of at least 128 cached rows, as many as keep about four blocks per SM busy
-                splits = max(1, min(16, -(-int(batch.max_kv_len) // 32) // 4))
+                reach = int(batch.max_kv_len) if not window else min(int(batch.max_kv_len), window + 32)
+                splits = max(1, min(16, -(-reach // 32) // 4))
                 while splits > 1 and batch.n_seqs * -(-n_head // 64) * splits > 4 * self.sm_count:
                     splits //= 2
                 if splits > 1:
                     scratch = torch.empty(T * n_head * splits * (dv + 2), dtype=torch.float32, device=q.device)
             return self._call("latent", "gfb_latent_attention", _ptr(q), _ptr(out), _ptr(kv.k_pool), _ptr(kv.page_table),
                               c_int(kv.page_table.shape[1]), c_int(kv.page_size), c_int(kv.k_pool.shape[0]), *self._batch_args(batch),
-                              c_int(int(batch.max_q_len)), c_int(n_head), c_int(head_dim), c_int(dv), c_float(scale), c_int(splits),
-                              _ptr(scratch), _ptr(batch.status), _stream())
+                              c_int(int(batch.max_q_len)), c_int(n_head), c_int(head_dim), c_int(dv), c_float(scale), c_int(window or 0),
+                              _ptr(sink), c_int(splits), _ptr(scratch), _ptr(batch.status), _stream())
         if (not values_in_keys and maps == 1 and dv == head_dim and q.dtype == torch.bfloat16 and kv.page_size == 64 and n_head // n_kv <= 8
                 and (head_dim in (64, 128) or (plain and head_dim % 8 == 0 and head_dim <= 256)) and (not (biased or capped) or scale > 0)
                 and not (keep_first and (biased or sink is not None))):

@@ -22,6 +22,7 @@ class BatchMeta:
     max_q_len: int                # host bound: longest run of new tokens
     max_kv_len: int               # host bound: longest sequence after this step
     status: torch.Tensor          # int32 [4], device-side error words
+    tokens: Optional[torch.Tensor] = None   # int32 [T], the step's token ids (for parts that read a per-token table)
 
 
 @dataclass

@@ -2,7 +2,7 @@
 
 A part is a small class that owns its parameters and launches kernels through
 `ops`; it takes its sizes and constants as constructor arguments and never
-sees the model's configuration.  Six kinds, one registry each:
+sees the model's configuration.  Eight kinds, one registry each:
 
     NORMS          forward(x32 [T,D], out [R,D], rows=None)
     POSITIONS      prepare(max_positions, device); what a mixer needs to place tokens
@@ -10,6 +10,8 @@ sees the model's configuration.  Six kinds, one registry each:
     FEED_FORWARDS  forward(h, residual)
     BLOCKS         roles; cache_needs(); forward(x32, batch, view, append): the arrangement of the above
     EMBEDDINGS     cache_needs(); forward(tokens, table, out, batch, view, scale): the token embedding plus something
+    TOKEN_INPUTS   forward(x, batch): what a layer adds to the stream for the token itself, from the model's side table
+    JUNCTIONS      forward(x, x0, turn): what happens to the stream ahead of a layer run that the schedule marks
 
 Every part also has `param_specs()` (name -> weights.loader.ParamSpec) and
 `load(tensors)`.  Mixers and feed-forwards ADD their result into `residual`, the
@@ -29,10 +31,12 @@ MIXERS: Dict[str, Callable] = {}
 FEED_FORWARDS: Dict[str, Callable] = {}
 BLOCKS: Dict[str, Callable] = {}
 EMBEDDINGS: Dict[str, Callable] = {}
+TOKEN_INPUTS: Dict[str, Callable] = {}
+JUNCTIONS: Dict[str, Callable] = {}
 
 # kind of part -> registry; a block arrangement names a kind for each of its roles
 REGISTRIES: Dict[str, Dict[str, Callable]] = {"norm": NORMS, "position": POSITIONS, "mixer": MIXERS,
-                                              "feed_forward": FEED_FORWARDS}
+                                              "feed_forward": FEED_FORWARDS, "token_input": TOKEN_INPUTS}
 
 
 def _registrar(table: Dict[str, Callable], kind: str):
@@ -53,6 +57,8 @@ register_mixer = _registrar(MIXERS, "mixer")
 register_feed_forward = _registrar(FEED_FORWARDS, "feed-forward")
 register_block = _registrar(BLOCKS, "block")
 register_embedding = _registrar(EMBEDDINGS, "embedding")
+register_token_input = _registrar(TOKEN_INPUTS, "token input")
+register_junction = _registrar(JUNCTIONS, "junction")
 
 
 def build_block(layer, dim: int, dtype, position):
@@ -87,4 +93,4 @@ def build_part(table: Dict[str, Callable], spec: PartSpec, **extra: Any):
 
 
 from . import norm, rope, attention, retention, feed_forward, block  # noqa: E402,F401  (register the built-in parts)
-from . import embedding, latent_attention, state_space, delta_rule, moe, mixer_sum, diff_attention, rglru  # noqa: E402,F401
+from . import embedding, latent_attention, state_space, delta_rule, moe, mixer_sum, diff_attention, rglru, gla, token_input, junction  # noqa: E402,F401

@@ -1,6 +1,7 @@
 """Arrangements of a layer's parts.  'prenorm' is gpt-fast's TransformerBlock
 (model.py:153-164): x += mixer(norm(x)); x += feed_forward(norm(x)), with the
-residual stream x kept in 32-bit.  'sandwich' norms a sublayer's output as well
+residual stream x kept in 32-bit, optionally with a learned factor per column on each
+sublayer and a token input behind them.  'sandwich' norms a sublayer's output as well
 and scales it before the sum; its feed-forward is optional.  'parallel' runs mixer and
 feed-forward side by side on two norms of the same x.
 
@@ -17,16 +18,29 @@ from .residual import Branch, as_residual
 
 @register_block("prenorm")
 class PreNormBlock:
-    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "ffn_norm": "norm"}
+    """x += s1 * mixer(norm1(x));  x += s2 * feed_forward(norm2(x));  then the token input, if the layer has one.
 
-    def __init__(self, parts: dict, dim: int, dtype: torch.dtype):
-        self.mixer, self.feed_forward = parts["mixer"], parts["feed_forward"]
-        self.mixer_norm, self.ffn_norm = parts["mixer_norm"], parts["ffn_norm"]
+    s1, s2: learned per-column factors (`layer_scale`; without it they are 1).  The feed-forward (with its norm) is optional.
+    A scaled sublayer writes into a `Branch` of its own and the scaled sum is left to the stream, whose next reader does it on
+    the way (`Residual.add_scaled`)."""
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "ffn_norm": "norm", "token_input": "token_input"}
+    optional_roles = ("feed_forward", "ffn_norm", "token_input")
+
+    def __init__(self, parts: dict, dim: int, dtype: torch.dtype, layer_scale: bool = False):
+        if ("feed_forward" in parts) != ("ffn_norm" in parts):
+            raise ValueError("a pre-norm block has a feed-forward with its norm or neither")
+        self._parts = dict(parts)
+        self.mixer, self.mixer_norm = parts["mixer"], parts["mixer_norm"]
+        self.feed_forward, self.ffn_norm, self.token_input = parts.get("feed_forward"), parts.get("ffn_norm"), parts.get("token_input")
         self.dim, self.dtype = dim, dtype
+        self.mixer_scale = self.ffn_scale = None
+        if layer_scale:
+            self.mixer_scale = self._parts["mixer_scale"] = LayerScale(dim)
+            if self.feed_forward is not None:
+                self.ffn_scale = self._parts["ffn_scale"] = LayerScale(dim)
 
     def parts(self):
-        return {"mixer": self.mixer, "feed_forward": self.feed_forward,
-                "mixer_norm": self.mixer_norm, "ffn_norm": self.ffn_norm}
+        return dict(self._parts)
 
     def cache_needs(self):
         """What one run of this layer keeps per sequence (its mixer's keys/values or state)."""
@@ -37,9 +51,18 @@ class PreNormBlock:
         x = as_residual(x)
         h = torch.empty(x.x.shape[0], self.dim, dtype=self.dtype, device=x.x.device)
         self.mixer_norm.forward(x, h)
-        self.mixer.forward(h, batch, view, residual=x, append=append)
-        self.ffn_norm.forward(x, h)
-        self.feed_forward.forward(h, residual=x)
+        y = x if self.mixer_scale is None else Branch(x.x.shape[0], self.dim, x.x.device)
+        self.mixer.forward(h, batch, view, residual=y, append=append)
+        if self.mixer_scale is not None:
+            x.add_scaled(y, self.mixer_scale.weight)
+        if self.feed_forward is not None:
+            self.ffn_norm.forward(x, h)
+            y = x if self.ffn_scale is None else Branch(x.x.shape[0], self.dim, x.x.device)
+            self.feed_forward.forward(h, residual=y)
+            if self.ffn_scale is not None:
+                x.add_scaled(y, self.ffn_scale.weight)
+        if self.token_input is not None:
+            self.token_input.forward(x, batch)
 
 
 @register_block("sandwich")

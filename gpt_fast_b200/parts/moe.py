@@ -11,6 +11,12 @@ the chosen experts by the softmax over just their logits (times scale).  `shared
 plain SwiGLU that every token runs; with `shared_gate` its output is multiplied by sigmoid(w_s . h), one number per token,
 whose row rides behind the router's rows in one product.
 
+Score 'softmax' takes s = softmax(z) over all experts, chooses by s + correction and weighs by s * scale as it is.
+`groups` = (count, keep): the experts are `count` equal groups of neighbours; a group's score is the largest choice score in it
+and only experts of the `keep` best groups can be chosen.  `activation` 'relu2': experts (and the shared one) of two products,
+W_down max(W_up h, 0)^2.  A shared expert without a gate and of the experts' own size is one more expert that every token
+chooses with weight 1, so the experts' products run it along; of another size it is a feed-forward of its own.
+
 The experts have no biases.  Their gate and up rows alternate in one matrix per expert, so one product yields both and
 applies the activation before anything is written; the weighted sum of the chosen experts' outputs is added to the
 residual stream in 32-bit by the kernel that does the down products (or by the one behind it)."""
@@ -19,7 +25,7 @@ import torch
 from .. import ops
 from ..weights.loader import ParamSpec
 from . import register_feed_forward
-from .residual import as_residual
+from .residual import Branch, as_residual
 
 
 def _pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
@@ -31,14 +37,22 @@ def _pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
 class MixtureOfExperts:
     def __init__(self, dim: int, hidden: int, n_experts: int, top: int, dtype: torch.dtype, router_scale: float = 1.0,
                  limit: float = 0.0, alpha: float = 1.0, shift: float = 0.0, correction: bool = True, score: str = "sigmoid",
-                 shared_hidden: int = 0, shared_gate: bool = False):
+                 shared_hidden: int = 0, shared_gate: bool = False, activation: str = "glu", groups=None):
         if not 1 <= top <= n_experts:
             raise ValueError(f"{top} of {n_experts} experts per token")
-        if score not in ("sigmoid", "softmax_top"):
-            raise ValueError(f"a router score is 'sigmoid' or 'softmax_top', not {score!r}")
+        if score not in ("sigmoid", "softmax_top", "softmax"):
+            raise ValueError(f"a router score is 'sigmoid', 'softmax_top' or 'softmax', not {score!r}")
+        if activation not in ("glu", "relu2"):
+            raise ValueError(f"the experts' activation is 'glu' or 'relu2', not {activation!r}")
+        if groups is not None and (groups[0] < 1 or n_experts % groups[0] or not 1 <= groups[1] <= groups[0]
+                                   or top > groups[1] * (n_experts // groups[0])):
+            raise ValueError(f"{top} experts from {groups[1]} of {groups[0]} groups of {n_experts} experts in all")
+        self.activation, self.groups = activation, None if groups is None or groups[0] == 1 else (int(groups[0]), int(groups[1]))
         if shared_gate and not shared_hidden:
             raise ValueError("a gate for a shared expert that is not there")
         self.score, self.shared_hidden, self.shared_gate = score, int(shared_hidden or 0), bool(shared_gate)
+        # one more expert that every token chooses, in the experts' own stacks
+        self.shared_inside = bool(self.shared_hidden) and not self.shared_gate and activation == "relu2" and self.shared_hidden == hidden
         self.shared_w13 = self.shared_w2 = None
         self.dim, self.hidden, self.n_experts, self.top, self.dtype = dim, hidden, int(n_experts), int(top), dtype
         self.router_scale, self.limit, self.alpha, self.shift = float(router_scale), float(limit), float(alpha), float(shift)
@@ -47,12 +61,16 @@ class MixtureOfExperts:
 
     def param_specs(self):
         E, F, D = self.n_experts, self.hidden, self.dim
-        specs = {"router": ParamSpec((E, D)), "gate": ParamSpec((E, F, D)), "up": ParamSpec((E, F, D)), "down": ParamSpec((E, D, F))}
+        specs = {"router": ParamSpec((E, D)), "up": ParamSpec((E, F, D)), "down": ParamSpec((E, D, F))}
+        if self.activation == "glu":
+            specs["gate"] = ParamSpec((E, F, D))
         if self.has_correction:
             specs["correction"] = ParamSpec((E,), "vector")
         if self.shared_hidden:
             Fs = self.shared_hidden
-            specs.update(shared_gate=ParamSpec((Fs, D)), shared_up=ParamSpec((Fs, D)), shared_down=ParamSpec((D, Fs)))
+            specs.update(shared_up=ParamSpec((Fs, D)), shared_down=ParamSpec((D, Fs)))
+            if self.activation == "glu":
+                specs["shared_gate"] = ParamSpec((Fs, D))
             if self.shared_gate:
                 specs["shared_sg"] = ParamSpec((1, D))
         return specs
@@ -61,15 +79,34 @@ class MixtureOfExperts:
         E, F, D = self.n_experts, self.hidden, self.dim
         self._router_stored = tensors["router"]
         self.router = _pad_rows(torch.cat([tensors["router"], tensors["shared_sg"]]) if self.shared_gate else tensors["router"])
-        if self.shared_hidden:
+        if self.shared_hidden and self.activation == "relu2":
+            self.shared_w13, self.shared_w2 = tensors["shared_up"], tensors["shared_down"]
+        elif self.shared_hidden:
             self.shared_w13 = torch.stack([tensors["shared_gate"], tensors["shared_up"]], dim=1).reshape(2 * self.shared_hidden, D).contiguous()
             self.shared_w2 = tensors["shared_down"]
         self.correction = tensors["correction"] if self.has_correction else torch.zeros(E, dtype=torch.float32, device=tensors["router"].device)
+        if self.activation == "relu2":
+            self.w13, self.w2 = tensors["up"], tensors["down"]
+            if self.shared_inside:
+                self.w13, self.w2 = torch.cat([self.w13, self.shared_w13[None]]), torch.cat([self.w2, self.shared_w2[None]])
+                self.shared_w13 = self.shared_w2 = None
+            return
         # rows alternate gate, up within every expert
         self.w13 = torch.stack([tensors["gate"], tensors["up"]], dim=2).reshape(E, 2 * F, D).contiguous()
         self.w2 = tensors["down"]
 
     def export(self):
+        if self.activation == "relu2":
+            E = self.n_experts
+            out = {"router": self._router_stored, "up": self.w13[:E], "down": self.w2[:E]}
+            if self.has_correction:
+                out["correction"] = self.correction
+            if self.shared_hidden:
+                out.update(shared_up=self.w13[E] if self.shared_inside else self.shared_w13,
+                           shared_down=self.w2[E] if self.shared_inside else self.shared_w2)
+                if self.shared_gate:
+                    out["shared_sg"] = self.router[E:E + 1]
+            return out
         w = self.w13.view(self.n_experts, self.hidden, 2, self.dim)
         out = {"router": self._router_stored, "gate": w[:, :, 0], "up": w[:, :, 1], "down": self.w2}
         if self.has_correction:
@@ -83,19 +120,20 @@ class MixtureOfExperts:
 
     def forward(self, h, residual):
         T = h.shape[0]
-        idx = torch.empty(T, self.top, dtype=torch.int32, device=h.device)
-        w = torch.empty(T, self.top, dtype=torch.float32, device=h.device)
-        if self.score == "sigmoid" and not self.shared_gate:
-            gate = ops.moe_router(h, self.router, self.correction, self.top, self.router_scale, idx, w)
-        else:
-            gate = ops.moe_router(h, self.router, self.correction, self.top, self.router_scale, idx, w, score=self.score,
-                                  n_extra=1 if self.shared_gate else 0)
+        slots = self.top + (1 if self.shared_inside else 0)
+        idx = torch.empty(T, slots, dtype=torch.int32, device=h.device)
+        w = torch.empty(T, slots, dtype=torch.float32, device=h.device)
+        gate = ops.moe_router(h, self.router, self.correction, self.top, self.router_scale, idx, w, score=self.score,
+                              n_extra=1 if self.shared_gate else 0, groups=self.groups, shared=self.shared_inside)
         residual = as_residual(residual)
-        x = residual.tensor()                                  # complete: the experts' kernel adds into it
-        ops.moe_experts(h, idx, w, self.w13, self.w2, x, self.limit, self.alpha, self.shift)
-        if self.shared_hidden:
+        x = residual.fresh() if isinstance(residual, Branch) else None       # an empty branch: the experts' kernel writes all of it
+        store = x is not None
+        if not store:
+            x = residual.tensor()                              # complete: the experts' kernel adds into it
+        ops.moe_experts(h, idx, w, self.w13, self.w2, x, self.limit, self.alpha, self.shift, act=self.activation, store=store)
+        if self.shared_hidden and not self.shared_inside:
             act = torch.empty(T, self.shared_hidden, dtype=self.dtype, device=h.device)
-            ops.linear(h, self.shared_w13, act, mode="swiglu")
+            ops.linear(h, self.shared_w13, act, mode="swiglu" if self.activation == "glu" else "relu2")
             if self.shared_gate:
                 # a factor per token commutes with the down product: it goes onto the activations
                 ops.sigmoid_gate(act, gate[0], gate[1], self.shared_hidden)

@@ -9,6 +9,14 @@ from . import register_norm
 from .residual import Residual
 
 
+def _owed_scaled(x: Residual, rows):
+    """The scaled branches a stream still owes, as the kernel that norms its rows takes them (at most two addends), if that
+    is all it owes; else None."""
+    if not x.scaled or rows is not None or x.pending is not None or x.normed is not None:
+        return None
+    return x.take_scaled(2)
+
+
 def _owed_rms_branch(x: Residual, rows):
     """The normed branch a stream still owes, as the norm kernel takes it, if one kernel can add it on its way (the
     branch's norm is a root-mean-square norm, no rows are gathered, nothing else is pending); else None."""
@@ -41,11 +49,14 @@ class RMSNorm:
         """x: the residual stream (a `Residual`, or a complete float32 tensor
         [T, dim]) -> out [R, dim] in the compute dtype; `rows` (int32 [R]) picks
         input rows, else R = T.  Partial sums pending on the stream are added
-        by the same kernel, and so is a branch with a root-mean-square norm of its own."""
+        by the same kernel, and so are a branch with a root-mean-square norm of its own or scaled branches."""
         if isinstance(x, Residual):
             branch = _owed_rms_branch(x, rows)
+            scaled = _owed_scaled(x, rows) if branch is None else None
             if branch is not None:
                 ops.layernorm(x.x, self.weight, None, self.eps, out, None, branch=branch, rms=True)
+            elif scaled is not None:
+                ops.layernorm_multi(x.x, scaled, [(self.weight, self.eps, out)], rms=True)
             else:
                 ops.rmsnorm(x.x, self.weight, self.eps, out, rows, x.take_pending())
         else:
@@ -77,8 +88,11 @@ class NoNorm:
     def forward(self, x, out, rows=None):
         if isinstance(x, Residual):
             branch = _owed_rms_branch(x, rows)
+            scaled = _owed_scaled(x, rows) if branch is None else None
             if branch is not None:
                 ops.layernorm(x.x, None, None, 0.0, out, None, branch=branch, rms=True)
+            elif scaled is not None:
+                ops.layernorm_multi(x.x, scaled, [(None, 0.0, out)], rms=True)
             else:
                 ops.layernorm(x.tensor(), None, None, 0.0, out, rows, rms=True)
         else:
@@ -141,13 +155,12 @@ class LayerNorm:
         are without bias."""
         if self.has_bias or other.has_bias:
             raise ValueError("two norms of one row in one kernel: only for norms without bias")
-        owed = x.take_scaled()
+        owed = x.take_scaled(2)
         pending = x.take_pending()
         if pending is not None:
+            if len(owed) == 2:
+                ops.layernorm_multi(x.x, owed[:1])
+                owed = owed[1:]
             owed = owed + [(pending, None)]
-        if len(owed) > 2:
-            x.scaled = owed[2:]
-            x.resolve()
-            owed = owed[:2]
-        ops.layernorm_multi(x.x, [(b if torch.is_tensor(b) else b.value(), s) for b, s in owed],
+        ops.layernorm_multi(x.x, owed,
                             [(self.weight, self.eps, out), (other.weight, other.eps, other_out)])

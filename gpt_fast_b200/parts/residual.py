@@ -32,9 +32,7 @@ class Residual:
 
     def resolve(self) -> None:
         if self.scaled:
-            owed, self.scaled = self.scaled, []
-            for i in range(0, len(owed), 2):
-                ops.layernorm_multi(self.x, [(b.value(), s) for b, s in owed[i:i + 2]])
+            self.take_scaled(0)
         if self.normed is not None:
             branch, norm, mult = self.take_normed()
             norm.add_into(self.x, branch, mult)
@@ -64,9 +62,17 @@ class Residual:
             self.resolve()
         self.scaled.append((branch, scale))
 
-    def take_scaled(self):
-        s, self.scaled = self.scaled, []
-        return s
+    def take_scaled(self, limit=None):
+        """The scaled branches still owed as (tensor or partial sums, factor) pairs, every addend of a branch a pair of its
+        own.  With more than `limit` of them the surplus (the first ones) is added here."""
+        owed, self.scaled = self.scaled, []
+        flat = [(v, s) for b, s in owed for v in (b.values() if isinstance(b, Branch) else [b])]
+        if limit is not None:
+            while len(flat) > limit:
+                n = min(2, len(flat) - limit)
+                ops.layernorm_multi(self.x, flat[:n])
+                flat = flat[n:]
+        return flat
 
     def take_normed(self):
         n, self.normed = self.normed, None
@@ -75,9 +81,7 @@ class Residual:
     def take_pending(self):
         """The partial sums still owed to x (the caller adds them); a normed or scaled branch is added first."""
         if self.scaled:
-            owed, self.scaled = self.scaled, []
-            for i in range(0, len(owed), 2):
-                ops.layernorm_multi(self.x, [(b.value(), s) for b, s in owed[i:i + 2]])
+            self.take_scaled(0)
         if self.normed is not None:
             branch, norm, mult = self.take_normed()
             norm.add_into(self.x, branch, mult)
@@ -118,6 +122,21 @@ class Branch(Residual):
     def resolve(self) -> None:
         self._materialise()
         super().resolve()
+
+    def fresh(self):
+        """The branch's tensor for a kernel that writes all of it, while the branch is still empty; else None."""
+        if not self.empty:
+            return None
+        self.empty = False
+        return self.x
+
+    def values(self):
+        """The addends of the branch as the kernels take them: complete float32 [T, dim] tensors or partial sums [S, T, dim],
+        one or two."""
+        if self.partials is None and self.pending is not None and not self.empty and self.normed is None and not self.scaled:
+            p, self.pending = self.pending, None
+            return [self.x, p]
+        return [self.value()]
 
     def value(self) -> torch.Tensor:
         """The branch as the norm kernels take it: the complete float32 [T, dim] tensor, or partial sums [S, T, dim]."""

@@ -81,32 +81,44 @@ class PlainOps:
         y.copy_((y.double() * g).to(y.dtype))
 
     # -- mixture of experts ---------------------------------------------------------------------
-    def moe_route(self, logits, correction, top, scale, idx, weights, score="sigmoid"):
+    def moe_route(self, logits, correction, top, scale, idx, weights, score="sigmoid", groups=(1, 1), shared=False):
         E = correction.shape[0]
-        s = torch.sigmoid(logits[:, :E].float()) if score == "sigmoid" else logits[:, :E].float()
+        z = logits[:, :E].float()
+        s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z.double(), -1).float() if score == "softmax" else z
         choice = s + correction.float()
+        per = E // groups[0]
+        if shared:
+            idx[:, top], weights[:, top] = E, 1.0
+            idx, weights = idx[:, :top], weights[:, :top]
         for t in range(s.shape[0]):
-            order = sorted(range(E), key=lambda e: (-float(choice[t, e]), e))[:top]
+            best = [float(choice[t, g * per:(g + 1) * per].max()) for g in range(groups[0])]
+            kept = set(sorted(range(groups[0]), key=lambda g: (-best[g], g))[:groups[1]])
+            order = sorted((e for e in range(E) if e // per in kept), key=lambda e: (-float(choice[t, e]), e))[:top]
             picked = s[t, order]
             idx[t] = torch.tensor(order, dtype=idx.dtype)
-            if score == "sigmoid":
+            if score == "softmax":
+                weights[t] = picked * scale
+            elif score == "sigmoid":
                 weights[t] = picked / (picked.sum() + 1e-20) * scale
             else:
                 weights[t] = torch.softmax(picked.double(), -1).float() * scale
 
-    def moe_experts(self, h, idx, weights, w13, w2, x, limit, alpha, shift=1.0):
+    def moe_experts(self, h, idx, weights, w13, w2, x, limit, alpha, shift=1.0, act="glu", store=False):
         hd = h.double()
         for t in range(h.shape[0]):
             acc = torch.zeros(x.shape[1], dtype=torch.float64)
             for r in range(idx.shape[1]):
                 e = int(idx[t, r])
                 z = w13[e].double() @ hd[t]
+                if act == "relu2":
+                    acc += float(weights[t, r]) * (w2[e].double() @ (torch.clamp(z, min=0) ** 2).to(h.dtype).double())
+                    continue
                 g, u = z[0::2], z[1::2]
                 if limit > 0:
                     g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
                 a = (g * torch.sigmoid(alpha * g) * (u + shift)).to(h.dtype).double()
                 acc += float(weights[t, r]) * (w2[e].double() @ a)
-            x[t] = (x[t].double() + acc).float()
+            x[t] = (acc if store else x[t].double() + acc).float()
 
     def rmsnorm(self, x, weight, eps, out, rows=None, pending=None):
         if pending is not None:
@@ -151,6 +163,9 @@ class PlainOps:
             x.copy_((x.double() + (y if scale is None else y * scale.double())).float())
         for w, eps, out in outs:
             v = (x if rows is None else x[rows.long()]).double()
+            if w is None:
+                out.copy_(v.to(out.dtype))
+                continue
             dev = v if rms else v - v.mean(-1, keepdim=True)
             out.copy_((dev * torch.rsqrt((dev * dev).mean(-1, keepdim=True) + eps) * w.double()).to(out.dtype))
 
@@ -172,13 +187,16 @@ class PlainOps:
                 raise IndexError("token lands on a page the slot does not hold")
             kv.k_pool[page, 0, pos % kv.page_size] = torch.cat([c, kr], -1).to(kv.k_pool.dtype)
 
-    def headwise_linear(self, a, w, out, n_head, k, n, a_off=0, a_stride=None, out_off=0, out_stride=None, gate=None, gate_off=0):
+    def headwise_linear(self, a, w, out, n_head, k, n, a_off=0, a_stride=None, out_off=0, out_stride=None, gate=None, gate_off=0,
+                        gate_per_head=False):
         a_stride = k if a_stride is None else a_stride
         out_stride = n if out_stride is None else out_stride
         for h in range(n_head):
             x = a[:, a_off + h * a_stride:a_off + h * a_stride + k].double()
             y = x @ w[h].double()
-            if gate is not None:
+            if gate_per_head:
+                y = y * torch.sigmoid(gate[:, gate_off + h:gate_off + h + 1].double())
+            elif gate is not None:
                 y = y * torch.sigmoid(gate[:, gate_off + h * n:gate_off + (h + 1) * n].double())
             out[:, out_off + h * out_stride:out_off + h * out_stride + n] = y.to(out.dtype)
 
@@ -203,6 +221,32 @@ class PlainOps:
             out[cu[s]:cu[s + 1]] = (y / (1 + torch.exp(-y)) if act else y).float()
             if taps > 1:                                           # one tap carries nothing
                 state[slot, state_off:state_off + (taps - 1) * C] = seq[n:].reshape(-1).float()
+
+    def gla(self, src, offsets, rank, a2, bias, tau, state, state_off, norm, eps, out, batch, n_head, head_dim, v_head_dim, q_scale):
+        H, d, dv, T = n_head, head_dim, v_head_dim, batch.n_tokens
+        qo, ko, vo, lo, go = offsets
+        x = src.double()
+        q, k = x[:, qo:qo + H * d].reshape(T, H, d) * q_scale, x[:, ko:ko + H * d].reshape(T, H, d)
+        v, gate = x[:, vo:vo + H * dv].reshape(T, H, dv), x[:, go:go + H * dv]
+        z = x[:, lo:lo + rank] @ a2.double().T + bias.double()
+        a = torch.exp(torch.nn.functional.logsigmoid(z) / tau).view(T, H, d)
+        _, slots = token_positions(batch)
+        o = torch.empty(T, H, dv, dtype=torch.float64)
+        for t in range(T):
+            S = state[int(slots[t]), state_off:state_off + H * d * dv].double().view(H, d, dv)
+            S = a[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+            state[int(slots[t]), state_off:state_off + H * d * dv] = S.reshape(-1).float()
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps) * norm.double()
+        out.copy_((o.reshape(T, H * dv) * gate * torch.sigmoid(gate)).to(out.dtype))
+
+    def token_gate(self, z, tokens, table, off, out, status):
+        rows = table[tokens.long()][:, off:off + z.shape[1]].double()
+        out.copy_((self._unary(z.double(), "gelu_tanh") * rows).to(out.dtype))
+
+    def pass_entry(self, x, x0, step, cat, y):
+        cat.copy_(torch.cat([x, x0], -1).to(cat.dtype))
+        y.copy_(step.float().expand_as(y))
 
     def rglru(self, u, w_a, w_i, b_a, b_i, lam, decay_scale, y_src, y_off, y_bias, state, state_off, out, batch):
         T, C = u.shape
