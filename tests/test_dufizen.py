@@ -77,10 +77,33 @@ def plain(folder, tokens, with_first_close_call=False):
     return _plain_cache[key] if with_first_close_call else _plain_cache[key][0]
 
 
+_noise_cache = {}
+
+
+def noise(folder, tokens):
+    """How far rounding moves each row of logits, relative to their scale: the plain statement with the sublayers' inputs in
+    bfloat16 and every weight moved by up to half a bfloat16 step, the largest of three draws.  Some positions are far more
+    sensitive than others: the recurrence's read-out is normed per head, so at a sequence's first token a q.k close to zero
+    decides a head's sign."""
+    key = (folder, tuple(tokens))
+    if key not in _noise_cache:
+        with open(os.path.join(folder, "config.json")) as f:
+            cfg = json.load(f)
+        w, want = load_file(os.path.join(folder, "model.safetensors")), plain(folder, tokens)
+        rows = []
+        for seed in range(3):
+            g = torch.Generator().manual_seed(seed)
+            moved = {k: v.double() * (1 + 2 ** -9 * (2 * torch.rand(v.shape, generator=g, dtype=torch.float64) - 1)) for k, v in w.items()}
+            rows.append((pd.forward(cfg, moved, tokens, act=torch.bfloat16).float() - want).pow(2).mean(-1).sqrt())
+        _noise_cache[key] = torch.stack(rows).max(0).values / float(want.pow(2).mean().sqrt())
+    return _noise_cache[key]
+
+
 def judge(got, folder, tokens, rows, dtype, where):
     """32-bit: equal to rounding.  bfloat16: up to the sequence's first token at which a router's choice is a close call every
-    row within a few per cent of the logits' own scale; from there on (another expert moves that token, and the mixers carry it
-    on) half of the rows within 0.06 of it.  A wrong key, page or state moves the rows by about the scale."""
+    row within a few per cent of the logits' own scale, or within a few times what rounding does to that row; from there on
+    (another expert moves that token, and the mixers carry it on) half of the rows within 0.06 of the scale.  A wrong key, page or
+    state moves the rows by about the scale."""
     want, first_close = plain(folder, tokens, True)
     positions = torch.arange(len(tokens))[rows]
     want = want[rows]
@@ -90,11 +113,11 @@ def judge(got, folder, tokens, rows, dtype, where):
         assert float((got - want).abs().max()) <= 2e-4 * max(scale, 1.0), f"{where}: off by {float((got - want).abs().max()):.2e}, scale {scale:.2f}"
     else:
         per_row = (got - want).pow(2).mean(-1).sqrt() / scale
-        sure = per_row[positions < first_close]
-        if sure.numel():
-            assert float(sure.pow(2).mean().sqrt()) <= 0.04, f"{where}: rms error {float(sure.pow(2).mean().sqrt()):.4f} of the scale"
-            assert float(sure.max()) <= 0.1, f"{where}: a row is off by {float(sure.max()):.3f} of the scale ahead of any close call"
-        assert float(per_row.median()) <= 0.06, f"{where}: half of the rows are off by {float(per_row.median()):.3f} of the scale or more"
+        loose = 0.04 + 4 * noise(folder, tokens)[rows]
+        sure = positions < first_close
+        over = (per_row > loose) & sure
+        assert not bool(over.any()), f"{where}: rows {positions[over].tolist()[:5]} are off by {per_row[over].tolist()[:5]}, allowed {loose[over].tolist()[:5]}"
+        assert float(per_row.median()) <= 0.06 + float(noise(folder, tokens)[rows].median()), f"{where}: half of the rows are off by {float(per_row.median()):.3f} of the scale or more"
 
 
 def tokens_of(vocab, n, seed):
@@ -149,7 +172,7 @@ def test_the_stream_after_every_layer_run(folders, backend, name):
     want = []
     pd.forward(cfg, load_file(os.path.join(folders[name], "model.safetensors")), toks, want)
     assert len(kept) == len(want) == {"dufizen-tiny-a": 11, "dufizen-tiny-b": 3}[name]
-    sure = len(toks) if backend[1] == "float32" else max(1, plain(folders[name], toks, True)[1])
+    sure = len(toks) if backend[1] == "float32" else max(1, plain(folders[name], toks, True)[1])      # up to the first close call
     for i, got in enumerate(kept):
         tol = (1e-4 if backend[1] == "float32" else 0.03) * float(want[i].float().pow(2).mean().sqrt())
         assert float((got[:sure] - want[i][:sure].float()).pow(2).mean().sqrt()) <= tol, f"the stream behind run {i}"
