@@ -398,7 +398,7 @@ def design_bench(a, design):
     import gpt_fast_b200 as gf
     from gpt_fast_b200 import ops
     from gpt_fast_b200.config.registry import config_from_name
-    # design -> [(named size, layers to build or None for all, the model beside it: a label and a config from the size's own)]
+    # design -> [(named size, layers to build or None for all, the model beside it (or several): a label and a config from the size's own)]
     tables = {"lasezen": [("lasezen-1b", None, "llama", llama_twin), ("lasezen-7b", a.layers or 8, "llama", llama_twin)],
               # beside Gikepel: the library's other hybrid of attention and a recurrent mixer, at the same width, depth,
               # feed-forward size and vocabulary
@@ -414,6 +414,10 @@ def design_bench(a, design):
     # token (Tapupel: three routed and the shared one)
     tables["tapupel"] = [("tapupel-1b", a.layers, "lomusun", lambda cfg: dict(config_from_name("lomusun-1b"),
                                                                              layers=config_from_name("lomusun-1b")["layers"][:len(cfg["layers"])]))]
+    # beside Dufizen (16 runs of 12 layers): the library's other design of latent attention and a recurrence with a decay per key
+    # channel, and its other design of three routed experts and a shared one of 1792, both at the same width, depth and vocabulary
+    tables["dufizen"] = [("dufizen-1b", a.layers, "gikepel", lambda cfg: config_from_name("gikepel-1b"),
+                          "tapupel", lambda cfg: config_from_name("tapupel-1b"))]
     if design not in tables:
         print(f"bench.py: no size table for design '{design}'")
         return 2
@@ -422,12 +426,12 @@ def design_bench(a, design):
     out = {"design": design, "dtype": "bf16", "data": "synthetic", "peaks": pk, "sizes": []}
     lengths = tuple(int(x) for x in a.prefill_lengths.split(",")) if a.prefill_lengths else (512, 2048, 8192)
     with ClockSampler() as clocks:
-        for name, n_layers, twin_label, twin in tables[design]:
+        for name, n_layers, *twins in tables[design]:
             cfg = config_from_name(name)
             if n_layers:
                 cfg["layers"] = cfg["layers"][:n_layers]
             row = {"size": name, "layers": len(cfg["layers"]), "width": cfg["width"]}
-            for label, source in ((design, cfg), (twin_label, twin(cfg))):
+            for label, source in [(design, cfg)] + [(twins[i], twins[i + 1](cfg)) for i in range(0, len(twins), 2)]:
                 # each model in a process of its own: the two then do not share a CUDA context or an allocator
                 cmd = [sys.executable, os.path.abspath(__file__), "--design-model", json.dumps(source), "--design-label", label,
                        "--steps", str(a.steps), "--warmup", str(a.warmup), "--prefill-lengths", ",".join(str(x) for x in lengths)]
@@ -465,7 +469,7 @@ def main():
     ap.add_argument("--skip-configs", action="store_true", help="leave out the Llama-3.2-3B and Llama-2-13B sizes")
     ap.add_argument("--skip-shares", action="store_true", help="leave out the per-kernel shares")
     ap.add_argument("--design", default=None, help="instead of the default workload: prefill and decode of another design "
-                    "(lasezen, gikepel, lomusun, tapupel) at layer sizes of a real model, beside the library's closest other model at equal size")
+                    "(lasezen, gikepel, lomusun, tapupel, dufizen) at layer sizes of a real model, beside the library's closest other model at equal size")
     ap.add_argument("--design-model", default=None, help=argparse.SUPPRESS)       # one model of --design, run as a child process
     ap.add_argument("--design-label", default="model", help=argparse.SUPPRESS)
     ap.add_argument("--prefill-lengths", default=None, help="with --design: prompt lengths of the prefill rows (default 512,2048,8192)")

@@ -52,9 +52,13 @@ gla_decay_kernel(const T* __restrict__ src, int ld, int low_off, int rank, const
 #pragma unroll
     for (int i = 0; i < DEC_TOKENS; i++) acc[i] = 0.f;
     const T* row = a2 + (size_t)c * rank;
-#pragma unroll 4
+    constexpr int N = 16 / sizeof(T);                // numbers of a row per 16-byte load
+    const bool wide = rank % N == 0 && (reinterpret_cast<uintptr_t>(a2) & 15) == 0;
+    uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll 8
     for (int r = 0; r < rank; r++) {
-        const float w = gfb_to_f32(row[r]);
+        if (wide && r % N == 0) raw = *reinterpret_cast<const uint4*>(row + r);
+        const float w = gfb_to_f32(wide ? reinterpret_cast<const T*>(&raw)[r % N] : row[r]);
         const float4* l = reinterpret_cast<const float4*>(low + r * DEC_TOKENS);
 #pragma unroll
         for (int i = 0; i < DEC_TOKENS / 4; i++) {
@@ -72,8 +76,8 @@ gla_decay_kernel(const T* __restrict__ src, int ld, int low_off, int rank, const
 // ---------------------------------------------------------------- chunks side by side ----
 constexpr int PC = 64;           // tokens per chunk
 constexpr int SUB = 16;          // tokens per sub-chunk
-constexpr int VS = 64;           // value columns per block
 constexpr int THREADS = 256;
+// VS below: value columns per block, 64 or (heads that have them) 128; a thread owns VS / 64 groups of four columns, 64 apart
 
 struct ChunkWork { int seq, slot, t0, n; };
 
@@ -95,74 +99,88 @@ __device__ __forceinline__ bool chunk_work(const GfbBatch& b, int w, ChunkWork& 
     return false;
 }
 
-// 64 key channels at a time; thread (channel, sub-chunk) sums the decays of its 16 tokens, then thread (ty, tx) owns key
-// channels 4 ty .. + 3 and value columns 4 tx .. + 3 of the product
-template <typename T>
+// A block takes 64 key channels and VS value columns.  Thread (channel, sub-chunk) sums the decays of its 16 tokens, then thread
+// (ty, tx) owns key channels 4 ty .. + 3 and value columns 4 tx .. + 3 (+ 64) of the product.
+template <typename T, int VS>
 __global__ void __launch_bounds__(THREADS)
 gla_state_kernel(const T* __restrict__ src, int ld, int k_off, int v_off, const float* __restrict__ g, float* __restrict__ U,
                  float* __restrict__ chunk_decay, GfbBatch b, int H, int d, int dv) {
-    __shared__ __align__(16) float Kc[PC][64];
-    __shared__ __align__(16) float Vs[PC][VS];
-    __shared__ float tot[4][64];
+    constexpr int NG = VS / 64;
+    extern __shared__ __align__(16) float sm[];
+    float* Kc = sm;                                  // [PC][64]: k 2^(the decays behind the token)
+    float* Vs = Kc + PC * 64;                        // [PC][VS]
+    float* tot = Vs + PC * VS;                       // [4][64]
     gfb_pdl_launch();
     gfb_pdl_wait();
     ChunkWork c;
     if (!chunk_work(b, blockIdx.x, c)) return;
-    const int w = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VS;
+    const int slices = (dv + VS - 1) / VS;
+    const int w = blockIdx.x, h = blockIdx.y, v0 = ((int)blockIdx.z % slices) * VS, d0 = ((int)blockIdx.z / slices) * 64;
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int dd = tid & 63, sub = tid >> 6, ch = d0 + dd;
+    float gi[SUB], ki[SUB], sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < SUB; i++) {
+        const int j = sub * SUB + i;
+        const bool live = j < c.n && ch < d;
+        gi[i] = live ? g[(size_t)(c.t0 + j) * H * d + (size_t)h * d + ch] : 0.f;
+        ki[i] = live ? gfb_to_f32(src[(size_t)(c.t0 + j) * ld + k_off + h * d + ch]) : 0.f;
+    }
+#pragma unroll 8
     for (int e = tid; e < PC * VS; e += THREADS) {
         const int j = e / VS, v = e - j * VS;
-        Vs[j][v] = (j < c.n && v0 + v < dv) ? gfb_to_f32(src[(size_t)(c.t0 + j) * ld + v_off + h * dv + v0 + v]) : 0.f;
+        Vs[e] = (j < c.n && v0 + v < dv) ? gfb_to_f32(src[(size_t)(c.t0 + j) * ld + v_off + h * dv + v0 + v]) : 0.f;
     }
-    const int dd = tid & 63, sub = tid >> 6;
-    float* Ug = U + ((size_t)w * H + h) * d * dv;
-    for (int d0 = 0; d0 < d; d0 += 64) {
-        const int ch = d0 + dd;
-        float gi[SUB], ki[SUB], sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < SUB; i++) {
-            const int j = sub * SUB + i;
-            const bool live = j < c.n && ch < d;
-            gi[i] = live ? g[(size_t)(c.t0 + j) * H * d + (size_t)h * d + ch] : 0.f;
-            ki[i] = live ? gfb_to_f32(src[(size_t)(c.t0 + j) * ld + k_off + h * d + ch]) : 0.f;
-            sum += gi[i];
-        }
-        __syncthreads();                            // the previous channels' product is done with Kc and tot
-        tot[sub][dd] = sum;
-        __syncthreads();
-        float after = 0.f;                           // decays behind this sub-chunk
-        for (int m = 3; m > sub; m--) after += tot[m][dd];
-        if (blockIdx.z == 0 && sub == 0 && ch < d) chunk_decay[((size_t)w * H + h) * d + ch] = exp2f(after + sum);
-        float behind = 0.f;                          // decays behind token i within the sub-chunk
+    for (int i = 0; i < SUB; i++) sum += gi[i];
+    tot[sub * 64 + dd] = sum;
+    __syncthreads();
+    float after = 0.f;                               // decays behind this sub-chunk
+    for (int m = 3; m > sub; m--) after += tot[m * 64 + dd];
+    if (v0 == 0 && sub == 0 && ch < d) chunk_decay[((size_t)w * H + h) * d + ch] = exp2f(after + sum);
+    float behind = 0.f;                              // decays behind token i within the sub-chunk
 #pragma unroll
-        for (int i = SUB - 1; i >= 0; i--) {
-            Kc[sub * SUB + i][dd] = ki[i] * exp2f(behind + after);
-            behind += gi[i];
-        }
-        __syncthreads();
-        float acc[4][4];
+    for (int i = SUB - 1; i >= 0; i--) {
+        Kc[(sub * SUB + i) * 64 + dd] = ki[i] * exp2f(behind + after);
+        behind += gi[i];
+    }
+    __syncthreads();
+    float acc[NG][4][4];
+#pragma unroll
+    for (int n = 0; n < NG; n++)
 #pragma unroll
         for (int r = 0; r < 4; r++)
 #pragma unroll
-            for (int cc = 0; cc < 4; cc++) acc[r][cc] = 0.f;
+            for (int cc = 0; cc < 4; cc++) acc[n][r][cc] = 0.f;
 #pragma unroll 4
-        for (int j = 0; j < c.n; j++) {
-            const float4 k4 = *reinterpret_cast<const float4*>(&Kc[j][4 * ty]);
-            const float4 v4 = *reinterpret_cast<const float4*>(&Vs[j][4 * tx]);
-            const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, vv[4] = {v4.x, v4.y, v4.z, v4.w};
+    for (int j = 0; j < c.n; j++) {
+        const float4 k4 = *reinterpret_cast<const float4*>(Kc + j * 64 + 4 * ty);
+        const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+        for (int n = 0; n < NG; n++) {
+            const float4 v4 = *reinterpret_cast<const float4*>(Vs + j * VS + 64 * n + 4 * tx);
+            const float vv[4] = {v4.x, v4.y, v4.z, v4.w};
 #pragma unroll
             for (int r = 0; r < 4; r++)
 #pragma unroll
-                for (int cc = 0; cc < 4; cc++) acc[r][cc] = fmaf(kk[r], vv[cc], acc[r][cc]);
+                for (int cc = 0; cc < 4; cc++) acc[n][r][cc] = fmaf(kk[r], vv[cc], acc[n][r][cc]);
         }
+    }
+    float* Ug = U + ((size_t)w * H + h) * d * dv;
+    const bool wide = dv % 4 == 0;                    // (U is 16-byte aligned)
 #pragma unroll
-        for (int r = 0; r < 4; r++) {
-            const int row = d0 + 4 * ty + r;
-            if (row >= d) continue;
+    for (int r = 0; r < 4; r++) {
+        const int row = d0 + 4 * ty + r;
+        if (row >= d) continue;
 #pragma unroll
-            for (int cc = 0; cc < 4; cc++) {
-                const int v = v0 + 4 * tx + cc;
-                if (v < dv) Ug[(size_t)row * dv + v] = acc[r][cc];
+        for (int n = 0; n < NG; n++) {
+            const int v = v0 + 64 * n + 4 * tx;
+            if (wide && v < dv) {
+                *reinterpret_cast<float4*>(Ug + (size_t)row * dv + v) = make_float4(acc[n][r][0], acc[n][r][1], acc[n][r][2], acc[n][r][3]);
+            } else {
+#pragma unroll
+                for (int cc = 0; cc < 4; cc++)
+                    if (v + cc < dv) Ug[(size_t)row * dv + v + cc] = acc[n][r][cc];
             }
         }
     }
@@ -184,17 +202,18 @@ gla_scan_kernel(float* __restrict__ U, const float* __restrict__ chunk_decay, fl
     const int row = (int)(e / dv);
     float* Sg = state + (size_t)b.slots[s] * state_ld + (size_t)h * per + e;
     float S = *Sg;
-    // four chunks' loads are in flight together
-    for (int c = 0; c < nc; c += 4) {
-        float add[4], dec[4];
+    // AHEAD chunks' loads are in flight together
+    constexpr int AHEAD = 16;
+    for (int c = 0; c < nc; c += AHEAD) {
+        float add[AHEAD], dec[AHEAD];
 #pragma unroll
-        for (int i = 0; i < 4; i++) {
+        for (int i = 0; i < AHEAD; i++) {
             const size_t at = (size_t)(first + min(c + i, nc - 1)) * H + h;
             add[i] = U[at * per + e];
             dec[i] = chunk_decay[at * d + row];
         }
 #pragma unroll
-        for (int i = 0; i < 4; i++)
+        for (int i = 0; i < AHEAD; i++)
             if (c + i < nc) {
                 U[((size_t)(first + c + i) * H + h) * per + e] = S;
                 S = fmaf(dec[i], S, add[i]);
@@ -204,26 +223,30 @@ gla_scan_kernel(float* __restrict__ U, const float* __restrict__ chunk_decay, fl
 }
 
 // Thread (ty, tx) of the 16 x 16 grid owns tokens ty + 16 r (one per sub-chunk, r = 0..3) against tokens tx + 16 c, and value
-// columns 4 tx .. + 3.  Key channels come DT at a time: q, k and L as they are, qt = q 2^L and kh = k 2^(L_end - L) for pairs in
+// columns 4 tx .. + 3 (+ 64).  Key channels come DT at a time: q, k and L as they are, qt = q 2^L and kh = k 2^(L_end - L) for pairs in
 // different sub-chunks.
 constexpr int DT = 32, DTP = DT + 4;
+template <int VS>
 struct OutSmem {
-    float q[PC][DTP], k[PC][DTP], L[PC][DTP], qt[PC][DTP], kh[PC][DTP];
+    union {
+        struct { float q[PC][DTP], k[PC][DTP], L[PC][DTP], qt[PC][DTP], kh[PC][DTP]; };
+        float A[PC][PC + 4];      // scores, lower triangle (behind the last pass)
+    };
     float S[DT][VS];              // the state ahead of the chunk, the channels of this pass
     float V[PC][VS];
-    float A[PC][PC + 4];          // scores, lower triangle
     float tot[8][DT];             // decay sums of half sub-chunks
     float M[4][DT];               // decay of a whole sub-chunk
 };
 
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 
-template <typename T>
+template <typename T, int VS>
 __global__ void __launch_bounds__(THREADS, 2)
 gla_out_kernel(const T* __restrict__ src, int ld, int q_off, int k_off, int v_off, const float* __restrict__ g, const float* __restrict__ U,
                float* __restrict__ out, GfbBatch b, int H, int d, int dv, float q_scale) {
+    constexpr int NG = VS / 64;
     extern __shared__ __align__(16) unsigned char raw[];
-    OutSmem& sm = *reinterpret_cast<OutSmem*>(raw);
+    OutSmem<VS>& sm = *reinterpret_cast<OutSmem<VS>*>(raw);
     gfb_pdl_launch();
     gfb_pdl_wait();
     ChunkWork c;
@@ -237,12 +260,16 @@ gla_out_kernel(const T* __restrict__ src, int ld, int q_off, int k_off, int v_of
     const float* Ug = U + ((size_t)w * H + h) * d * dv;
     float far[4][4];                                // scores of tokens in different sub-chunks: [r][c], c < r
     float near[4];                                  // scores within a sub-chunk: token ty against tx
-    float o[4][4];
+    float o[NG][4][4];
 #pragma unroll
     for (int r = 0; r < 4; r++) {
         near[r] = 0.f;
 #pragma unroll
-        for (int cc = 0; cc < 4; cc++) far[r][cc] = o[r][cc] = 0.f;
+        for (int cc = 0; cc < 4; cc++) {
+            far[r][cc] = 0.f;
+#pragma unroll
+            for (int n = 0; n < NG; n++) o[n][r][cc] = 0.f;
+        }
     }
     const int dd = tid & 31, oct = tid >> 5;        // staging: a channel, eight tokens
     for (int d0 = 0; d0 < d; d0 += DT) {
@@ -316,19 +343,24 @@ gla_out_kernel(const T* __restrict__ src, int ld, int q_off, int k_off, int v_of
             const float p1[4] = {M0.x, M0.y, M0.z, M0.w}, m1[4] = {M1.x, M1.y, M1.z, M1.w}, m2[4] = {M2.x, M2.y, M2.z, M2.w};
 #pragma unroll
             for (int y = 0; y < 4; y++) {
-                const float4 s4 = ld4(&sm.S[x + y][4 * tx]);
                 const float p2 = p1[y] * m1[y], p3 = p2 * m2[y];
-                const float e0 = y == 0 ? qt[0].x : y == 1 ? qt[0].y : y == 2 ? qt[0].z : qt[0].w;
-                const float e1 = (y == 0 ? qt[1].x : y == 1 ? qt[1].y : y == 2 ? qt[1].z : qt[1].w) * p1[y];
-                const float e2 = (y == 0 ? qt[2].x : y == 1 ? qt[2].y : y == 2 ? qt[2].z : qt[2].w) * p2;
-                const float e3 = (y == 0 ? qt[3].x : y == 1 ? qt[3].y : y == 2 ? qt[3].z : qt[3].w) * p3;
-                o[0][0] = fmaf(e0, s4.x, o[0][0]); o[0][1] = fmaf(e0, s4.y, o[0][1]); o[0][2] = fmaf(e0, s4.z, o[0][2]); o[0][3] = fmaf(e0, s4.w, o[0][3]);
-                o[1][0] = fmaf(e1, s4.x, o[1][0]); o[1][1] = fmaf(e1, s4.y, o[1][1]); o[1][2] = fmaf(e1, s4.z, o[1][2]); o[1][3] = fmaf(e1, s4.w, o[1][3]);
-                o[2][0] = fmaf(e2, s4.x, o[2][0]); o[2][1] = fmaf(e2, s4.y, o[2][1]); o[2][2] = fmaf(e2, s4.z, o[2][2]); o[2][3] = fmaf(e2, s4.w, o[2][3]);
-                o[3][0] = fmaf(e3, s4.x, o[3][0]); o[3][1] = fmaf(e3, s4.y, o[3][1]); o[3][2] = fmaf(e3, s4.z, o[3][2]); o[3][3] = fmaf(e3, s4.w, o[3][3]);
+                const float e[4] = {y == 0 ? qt[0].x : y == 1 ? qt[0].y : y == 2 ? qt[0].z : qt[0].w,
+                                    (y == 0 ? qt[1].x : y == 1 ? qt[1].y : y == 2 ? qt[1].z : qt[1].w) * p1[y],
+                                    (y == 0 ? qt[2].x : y == 1 ? qt[2].y : y == 2 ? qt[2].z : qt[2].w) * p2,
+                                    (y == 0 ? qt[3].x : y == 1 ? qt[3].y : y == 2 ? qt[3].z : qt[3].w) * p3};
+#pragma unroll
+                for (int n = 0; n < NG; n++) {
+                    const float4 s4 = ld4(&sm.S[x + y][64 * n + 4 * tx]);
+#pragma unroll
+                    for (int r = 0; r < 4; r++) {
+                        o[n][r][0] = fmaf(e[r], s4.x, o[n][r][0]); o[n][r][1] = fmaf(e[r], s4.y, o[n][r][1]);
+                        o[n][r][2] = fmaf(e[r], s4.z, o[n][r][2]); o[n][r][3] = fmaf(e[r], s4.w, o[n][r][3]);
+                    }
+                }
             }
         }
     }
+    __syncthreads();                                 // the scores take the place of q, k, L
     // scores to shared memory: row ty + 16 r, column tx + 16 c (columns of later sub-chunks are never read)
 #pragma unroll
     for (int r = 0; r < 4; r++) {
@@ -342,12 +374,17 @@ gla_out_kernel(const T* __restrict__ src, int ld, int q_off, int k_off, int v_of
         if (16 * J >= c.n) break;                    // uniform: no tokens there
 #pragma unroll 4
         for (int jj = 0; jj < SUB; jj++) {
-            const float4 v4 = ld4(&sm.V[16 * J + jj][4 * tx]);
+            float a[4];
 #pragma unroll
-            for (int r = J; r < 4; r++) {
-                const float a = sm.A[ty + 16 * r][16 * J + jj];
-                o[r][0] = fmaf(a, v4.x, o[r][0]); o[r][1] = fmaf(a, v4.y, o[r][1]);
-                o[r][2] = fmaf(a, v4.z, o[r][2]); o[r][3] = fmaf(a, v4.w, o[r][3]);
+            for (int r = J; r < 4; r++) a[r] = sm.A[ty + 16 * r][16 * J + jj];
+#pragma unroll
+            for (int n = 0; n < NG; n++) {
+                const float4 v4 = ld4(&sm.V[16 * J + jj][64 * n + 4 * tx]);
+#pragma unroll
+                for (int r = J; r < 4; r++) {
+                    o[n][r][0] = fmaf(a[r], v4.x, o[n][r][0]); o[n][r][1] = fmaf(a[r], v4.y, o[n][r][1]);
+                    o[n][r][2] = fmaf(a[r], v4.z, o[n][r][2]); o[n][r][3] = fmaf(a[r], v4.w, o[n][r][3]);
+                }
             }
         }
     }
@@ -355,10 +392,17 @@ gla_out_kernel(const T* __restrict__ src, int ld, int q_off, int k_off, int v_of
     for (int r = 0; r < 4; r++) {
         const int i = ty + 16 * r;
         if (i >= c.n) continue;
+        float* dst = out + ((size_t)(c.t0 + i) * H + h) * dv;
 #pragma unroll
-        for (int cc = 0; cc < 4; cc++) {
-            const int v = v0 + 4 * tx + cc;
-            if (v < dv) out[((size_t)(c.t0 + i) * H + h) * dv + v] = o[r][cc];
+        for (int n = 0; n < NG; n++) {
+            const int v = v0 + 64 * n + 4 * tx;
+            if (dv % 4 == 0 && v < dv) {              // (out is 16-byte aligned)
+                *reinterpret_cast<float4*>(dst + v) = make_float4(o[n][r][0], o[n][r][1], o[n][r][2], o[n][r][3]);
+            } else {
+#pragma unroll
+                for (int cc = 0; cc < 4; cc++)
+                    if (v + cc < dv) dst[v + cc] = o[n][r][cc];
+            }
         }
     }
 }
@@ -381,38 +425,44 @@ GFB_API int gfb_gla(const void* src, int dt, int ld, int q_off, int k_off, int v
     if (rank < 1 || H < 1 || d < 1 || dv < 1) return gfb_fail("gfb_gla: rank %d, %d heads of %d and %d", rank, H, d, dv);
     const int chunks = n_tokens / PC + n_seqs;                    // an upper bound; surplus blocks find no work
     const int C = H * d;
-    if (H > 65535 || n_seqs > 65535 || (dv + VS - 1) / VS > 65535 || (C + 127) / 128 > 65535)
+    const int vs = dv > 64 ? 128 : 64, slices = (dv + vs - 1) / vs, dtiles = (d + 63) / 64;
+    if (H > 65535 || n_seqs > 65535 || (long)slices * dtiles > 65535 || (C + 127) / 128 > 65535)
         return gfb_fail("gfb_gla: %d heads of %d and %d exceed the grid limit", H, d, dv);
     const size_t dsmem = (size_t)rank * DEC_TOKENS * sizeof(float);
     if (dsmem > 48 * 1024) return gfb_fail("gfb_gla: decays of rank %d do not fit shared memory", rank);
+    if (((uintptr_t)out | (uintptr_t)scratch) & 15) return gfb_fail("gfb_gla: output and scratch must be 16-byte aligned");
     GfbBatch b{cu_seqlens, tok_seq, slots, lengths, n_seqs, n_tokens};
     float* g = scratch;
     float* decay = g + ((long)n_tokens * C + 3) / 4 * 4;
     float* U = decay + ((long)chunks * C + 3) / 4 * 4;
-    const dim3 cgrid(chunks, H, (dv + VS - 1) / VS), dgrid((n_tokens + DEC_TOKENS - 1) / DEC_TOKENS, (C + 127) / 128);
+    const dim3 dgrid((n_tokens + DEC_TOKENS - 1) / DEC_TOKENS, (C + 127) / 128);
+    const size_t ssmem = ((size_t)PC * 64 + (size_t)PC * vs + 4 * 64) * sizeof(float);
     cudaError_t e;
-#define GO(T)                                                                                                                       \
+#define GO(T, V)                                                                                                                    \
     do {                                                                                                                            \
         static bool configured = false;                                                                                             \
         if (!configured) {                                                                                                          \
-            e = cudaFuncSetAttribute(gla_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(OutSmem));         \
+            e = cudaFuncSetAttribute(gla_out_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(OutSmem<V>));   \
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_state_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ssmem); \
             if (e != cudaSuccess) return gfb_fail("gfb_gla: %s", cudaGetErrorString(e));                                            \
             configured = true;                                                                                                      \
         }                                                                                                                           \
         e = gfb_launch(gla_decay_kernel<T>, dgrid, dim3(128), dsmem, stream, (const T*)src, ld, low_off, rank, (const T*)a2, bias, b_dt, \
                        factor, g, n_tokens, C);                                                                                     \
         if (e == cudaSuccess)                                                                                                       \
-            e = gfb_launch(gla_state_kernel<T>, cgrid, dim3(THREADS), 0, stream, (const T*)src, ld, k_off, v_off, (const float*)g, U, decay, \
-                           b, H, d, dv);                                                                                            \
+            e = gfb_launch(gla_state_kernel<T, V>, dim3(chunks, H, slices * dtiles), dim3(THREADS), ssmem, stream, (const T*)src, ld, k_off, \
+                           v_off, (const float*)g, U, decay, b, H, d, dv);                                                          \
         if (e == cudaSuccess)                                                                                                       \
             e = gfb_launch(gla_scan_kernel, dim3((unsigned)(((size_t)d * dv + 255) / 256), n_seqs, H), dim3(256), 0, stream, U,     \
                            (const float*)decay, state, (size_t)state_ld, b, H, d, dv);                                              \
         if (e == cudaSuccess)                                                                                                       \
-            e = gfb_launch(gla_out_kernel<T>, cgrid, dim3(THREADS), sizeof(OutSmem), stream, (const T*)src, ld, q_off, k_off, v_off, \
-                           (const float*)g, (const float*)U, out, b, H, d, dv, q_scale);                                            \
+            e = gfb_launch(gla_out_kernel<T, V>, dim3(chunks, H, slices), dim3(THREADS), sizeof(OutSmem<V>), stream, (const T*)src, ld, q_off, \
+                           k_off, v_off, (const float*)g, (const float*)U, out, b, H, d, dv, q_scale);                              \
     } while (0)
-    if (dt == GFB_BF16) GO(__nv_bfloat16);
-    else if (dt == GFB_F32) GO(float);
+    if (dt == GFB_BF16 && vs == 128) GO(__nv_bfloat16, 128);
+    else if (dt == GFB_BF16) GO(__nv_bfloat16, 64);
+    else if (dt == GFB_F32 && vs == 128) GO(float, 128);
+    else if (dt == GFB_F32) GO(float, 64);
     else return gfb_fail("gfb_gla: unknown type %d", dt);
 #undef GO
     return gfb_check(e, "gfb_gla");

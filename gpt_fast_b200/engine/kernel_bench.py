@@ -8,6 +8,7 @@ the small, self-ending workload that profiler captures are taken on.
     python -m gpt_fast_b200.engine.kernel_bench attention --batch 1 --context 0 --new 2048
     python -m gpt_fast_b200.engine.kernel_bench sample --batch 8 --vocab 128256
     python -m gpt_fast_b200.engine.kernel_bench experts --tokens 2048 --experts 16 --top 4 --ff 1792 --dim 2048
+    python -m gpt_fast_b200.engine.kernel_bench gla --tokens 2048 --heads 16 --head_dim 128 --v_dim 128
 
 Weights are cycled through enough copies to exceed the L2 cache, so a memory-
 bound kernel is timed against DRAM.  gpt-fast has no per-kernel timing; its
@@ -164,6 +165,26 @@ def bench_experts(a):
           f"{2.0 * T * top * 3 * F * D / total / 1e6:.0f} TFLOP/s, the {busy} chosen experts' weights at {busy * 3 * F * D * 2 / total / 1e3:.0f} GB/s")
 
 
+def bench_gla(a):
+    """Gated linear attention over one prompt (--batch 1) or a decode step (--tokens 1) of `batch` sequences."""
+    B, T, H, d, dv, rank = a.batch, a.tokens, a.heads, a.head_dim, a.v_dim, 16
+    meta, _ = paged_batch(B, 0, T, 1, 8)
+    W = 2 * H * d + 2 * H * dv + rank
+    src = torch.randn(B * T, W, device="cuda").bfloat16()
+    a2, bias = (torch.randn(H * d, rank, device="cuda") * 0.3).bfloat16(), torch.randn(H * d, device="cuda")
+    norm, out = torch.ones(dv, device="cuda"), torch.empty(B * T, H * dv, device="cuda", dtype=torch.bfloat16)
+    copies = max(1, int(2 * L2_BYTES // (B * H * d * dv * 4)) + 1) if T == 1 else 1
+    states = [torch.zeros(B, H * d * dv, device="cuda") for _ in range(copies)]
+    offs = (0, H * d, 2 * H * d, W - rank, 2 * H * d + H * dv)
+    us = graph_time_us(lambda i: ops.gla(src, offs, rank, a2, bias, 16.0, states[i % copies], 0, norm, 1e-5, out, meta, H, d, dv, d ** -0.5), a.reps)
+    if T == 1:
+        print(f"gla decode batch={B} heads={H} {d} x {dv}: {us:.1f} us, states at {2 * B * H * d * dv * 4 / us / 1e3:.0f} GB/s")
+    else:
+        flops = B * T * H * 4.0 * d * dv                      # the recurrence itself: the state's update and its read-out
+        print(f"gla prefill batch={B} tokens={T} heads={H} {d} x {dv}: {us:.1f} us, {flops / us / 1e6:.1f} TFLOP/s of the recurrence")
+    ops.check_status(meta.status)
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser(prog="kernel_bench")
     sub = ap.add_subparsers(dest="what", required=True)
@@ -193,8 +214,12 @@ def main(argv=None):
     p.add_argument("--top", type=int, default=4); p.add_argument("--ff", type=int, default=1792)
     p.add_argument("--dim", type=int, default=2048); p.add_argument("--limit", type=float, default=7.0)
     p.add_argument("--reps", type=int, default=5)
+    p = sub.add_parser("gla")
+    p.add_argument("--batch", type=int, default=1); p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--heads", type=int, default=16); p.add_argument("--head_dim", type=int, default=128)
+    p.add_argument("--v_dim", type=int, default=128); p.add_argument("--reps", type=int, default=10)
     a = ap.parse_args(argv)
-    {"experts": bench_experts, "linear": bench_linear, "attention": bench_attention, "sample": bench_sample, "norm": bench_norm}[a.what](a)
+    {"gla": bench_gla, "experts": bench_experts, "linear": bench_linear, "attention": bench_attention, "sample": bench_sample, "norm": bench_norm}[a.what](a)
     ops.check_status(ops.new_status("cuda"))
     return 0
 
