@@ -463,7 +463,7 @@ def random_config(seed):
             layers.append(_gla(pick(1, 2, 5), pick(4, 9, 16, 40), pick(3, 8, 36, 70), pick(0.7, 4.0, 16.0), pick(1, 8, 12), mlp))
         else:
             layers.append(_latent(pick(1, 3, 4), pick(5, 16, 32), pick(2, 8, 16), pick(4, 16, 21), pick(16, 30, 48, 64), pick(1, 2, 17, 64, 65, 300),
-                                  pick(0.1, 0.5), pick(100.0, 20000.0), mlp))
+                                  pick(0.1, 0.5), pick(100.0, 30000.0), mlp))
     cfg = {"architecture": "Dufizen", "vocab": pick(50, 97, 128), "width": pick(24, 37, 64), "norm": {"eps": pick(1e-6, 1e-3)},
            "token_side": {"dim": pick(1, 8, 11)}, "layers": layers}
     if pick(0, 1, 1):

@@ -191,7 +191,7 @@ def lat_case(m, seed, backend, s=0.3, sink=1.0):
 
 # the second and third shapes are those the tensor-core attention takes in bfloat16
 @pytest.mark.parametrize("m", [lat_m(), lat_m(H=4, d=16, r=16, dv=8, R=32, W=65), lat_m(H=5, d=8, r=16, dv=12, R=48, W=1),
-                               lat_m(H=1, d=7, r=2, dv=3, R=9, W=1000, base=20000.0), lat_m(H=2, d=16, r=16, dv=16, R=16, W=64)])
+                               lat_m(H=1, d=7, r=2, dv=3, R=9, W=1000, base=30000.0), lat_m(H=2, d=16, r=16, dv=16, R=16, W=64)])
 def test_latent_attention(backend, m):
     part, w = lat_case(m, 21, backend)
     seqs = [list(range(140)), list(range(140, 229))]
@@ -224,12 +224,12 @@ def loud_case(m, seed, backend, T, key, query):
 
 
 @pytest.mark.parametrize("shape", [dict(), dict(H=4, d=16, r=16, dv=8, R=32)])
-@pytest.mark.parametrize("W,key,query", [(19, 60, 78), (64, 63, 126), (65, 64, 128), (200, 3, 202), (5, 127, 131), (96, 40, 135)])
+@pytest.mark.parametrize("W,key,query", [(19, 60, 78), (64, 63, 126), (65, 64, 128), (200, 3, 202), (5, 127, 131), (100, 40, 135)])
 def test_the_windows_edge(backend, shape, W, key, query):
     """A loud key W - 1 positions back is seen, one position later it is gone: in a prompt, in portions whose borders fall
     between them, and in decode steps."""
     m = lat_m(W=W, scale=1.0, **shape)
-    assert query - key == W - 1 or W == 96
+    assert query - key == W - 1 or W == 100
     T = query + 4
     part, w, h = loud_case(m, 91, backend, T, key, query - 2 if W > 2 else query)
     want = pd.latent_attention(h.double(), f64(w), m, EPS)
@@ -289,7 +289,7 @@ def mlp_of(E, top, ff, groups=None, shared=None):
 
 
 @pytest.mark.parametrize("T", [1, 3, 20, 70, 300])
-@pytest.mark.parametrize("mlp", [mlp_of(12, 2, 16, (2, 1), 16), mlp_of(9, 4, 24, (3, 2), 40), mlp_of(5, 5, 11), mlp_of(40, 1, 8, (20, 3), 8),
+@pytest.mark.parametrize("mlp", [mlp_of(14, 3, 16, (2, 1), 16), mlp_of(9, 4, 24, (3, 2), 40), mlp_of(5, 5, 11), mlp_of(40, 1, 8, (20, 3), 8),
                                  mlp_of(6, 2, 13, (6, 2), 9)])
 def test_experts(backend, mlp, T):
     part, w = moe_case(mlp, 13, backend)
