@@ -166,3 +166,41 @@ def test_bad_token_is_reported_by_the_token_gate():
     with pytest.raises(ops.KernelError, match="token id out of range"):
         ops.check_status(st)
     assert out[1].abs().sum() == 0 and out[0].abs().sum() > 0
+
+
+# ---- nothing is written outside an output -----------------------------------------------------------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_new_kernels_stay_inside_their_outputs(dtype):
+    from test_kernels_canary_gpu import Guarded
+    H, rank = 3, 5
+    for q_lens, d, dv in (([1, 1], 33, 36), ([70, 1, 129], 33, 36), ([3, 64], 130, 71), ([65], 20, 130)):
+        batch, _, _ = make_batch(q_lens, [2] * len(q_lens), 3, 64, 4, seed=2)
+        T, C = batch.n_tokens, H * d
+        src = rnd(T, 2 * C + 2 * H * dv + rank, dtype=dtype, seed=1)
+        offs = (0, C, 2 * C, 2 * C + 2 * H * dv, 2 * C + H * dv)
+        state, out = Guarded(3, H * d * dv, fill=rnd(3, H * d * dv, seed=3)), Guarded(T, H * dv, dtype=dtype)
+        ops.gla(src, offs, rank, rnd(C, rank, dtype=dtype, seed=4), rnd(C, seed=5), 2.0, state.t, 0, rnd(dv, seed=6), 1e-5, out.t, batch, H, d, dv, 0.2)
+        state.check(f"gla state, {q_lens}")
+        out.check(f"gla, {q_lens}")
+    T, n, D, V = 13, 7, 44, 20
+    tokens = torch.randint(0, V, (T,), dtype=torch.int32, device=DEV)
+    g = Guarded(T, n, dtype=dtype)
+    ops.token_gate(rnd(T, n), tokens, rnd(V, 3 * n, dtype=dtype), 2 * n, g.t, ops.new_status(DEV))
+    g.check("token gate")
+    cat, y = Guarded(T, 2 * D, dtype=dtype), Guarded(T, D)
+    ops.pass_entry(rnd(T, D), rnd(T, D), rnd(D, dtype=dtype), cat.t, y.t)
+    cat.check("pass entry")
+    y.check("pass entry (the new stream)")
+    for T, F, D in ((1, 13, 21), (70, 13, 21), (9, 24, 40), (300, 40, 72)):
+        E, top = 5, 2
+        idx = torch.stack([torch.randperm(E)[:top] for _ in range(T)]).int().to(DEV)
+        x = Guarded(T, D)
+        ops.moe_experts(rnd(T, D, dtype=dtype), idx, torch.rand(T, top, device=DEV), rnd(E, F, D, dtype=dtype), rnd(E, D, F, dtype=dtype), x.t, 0.0, 1.0,
+                        0.0, act="relu2", store=True)
+        x.check(f"squared-ReLU experts, {T} tokens")
+    for T, E in ((5, 12), (200, 12)):
+        idx, w = Guarded(T, 4, dtype=torch.int32), Guarded(T, 4)
+        ops.moe_router(rnd(T, 24, dtype=dtype), rnd(16, 24, dtype=dtype, seed=2), rnd(E), 3, 1.0, idx.t, w.t, score="softmax", groups=(3, 2), shared=True)
+        idx.check("router's choice")
+        w.check("router's weights")
