@@ -65,6 +65,7 @@ class ModelSpec:
     embedding: Optional[PartSpec] = None  # what is added to the token embedding (a part of `parts.EMBEDDINGS`; None: nothing)
     junctions: List[PartSpec] = field(default_factory=list)   # parts of `parts.JUNCTIONS` that schedule entries name
     token_table: int = 0                  # columns of the per-token side table that layers' token inputs read (0: none)
+    streams: int = 0                      # residual streams per token (0: the one ordinary stream); every block then takes streams
     launch_overlap: bool = True           # kernels of a step may start while their predecessor drains; False: strictly in turn
 
     def validate(self) -> None:
@@ -72,6 +73,8 @@ class ModelSpec:
             raise ValueError(f"ModelSpec.logit_cap = {self.logit_cap}: a soft cap must be positive")
         if self.embed_scale is not None and self.embed_scale != self.embed_scale:
             raise ValueError("ModelSpec.embed_scale is not a number")
+        if self.streams < 0 or (self.streams and self.junctions):
+            raise ValueError(f"ModelSpec.streams = {self.streams}: not negative, and without junctions")
         owners = {}
         for i, e in enumerate(self.schedule):
             if not 0 <= e.layer < len(self.layers):

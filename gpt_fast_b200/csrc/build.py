@@ -40,6 +40,7 @@ LIBRARIES = {
     "recurrent": (["recurrent.cu"], [], []),
     "moe": (["moe.cu"], [], []),
     "gla": (["gla.cu"], [], []),
+    "streams": (["streams.cu"], [], []),
 }
 HEADERS = ["common.cuh", "attn_decode_noalloc.h"]
 

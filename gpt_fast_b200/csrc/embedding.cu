@@ -156,3 +156,46 @@ GFB_API int gfb_token_gate(const int* tokens, const void* side, int side_dt, int
 #undef GO
     return gfb_check(e, "gfb_token_gate");
 }
+
+// ---- token embedding behind a norm ---------------------------------------------------
+// out[t] = e / sqrt(mean(e^2) + eps) * w,  e = table[tokens[t]] * scale, 32-bit.  A block per token; a row is read twice (the second
+// time from L1).
+template <typename TW>
+__global__ void embed_normed_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, const void* __restrict__ w, int w_dt,
+                                    float* __restrict__ out, int D, int V, float scale, float eps, int* status) {
+    __shared__ float scratch[32];
+    gfb_pdl_launch();
+    gfb_pdl_wait();
+    const int t = blockIdx.x;
+    const int id = tokens[t];
+    float* o = out + (size_t)t * D;
+    if (id < 0 || id >= V) {
+        if (threadIdx.x == 0) gfb_report(status, GFB_ERR_TOKEN_RANGE, t, id);
+        for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = 0.f;
+        return;
+    }
+    const TW* e = table + (size_t)id * D;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) { const float v = gfb_to_f32(e[i]) * scale; ss += v * v; }
+    const float r = 1.0f / sqrtf(gfb_block_sum(ss, scratch) / (float)D + eps);
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+        const float g = w_dt == GFB_BF16 ? __bfloat162float(((const __nv_bfloat16*)w)[i]) : ((const float*)w)[i];
+        o[i] = gfb_to_f32(e[i]) * scale * r * g;
+    }
+}
+
+GFB_API int gfb_embed_normed(const int* tokens, const void* table, int table_dt, const void* w, int w_dt, float* out, int T, int D, int V,
+                             float scale, float eps, int* status, cudaStream_t stream) {
+    if (T <= 0 || D <= 0) return 0;
+    const int threads = D >= 1024 ? 256 : 128;
+    cudaError_t e;
+    if (table_dt == GFB_BF16)
+        e = gfb_launch(embed_normed_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, tokens, (const __nv_bfloat16*)table, w, w_dt, out, D, V,
+                       scale, eps, status);
+    else if (table_dt == GFB_F32)
+        e = gfb_launch(embed_normed_kernel<float>, dim3(T), dim3(threads), 0, stream, tokens, (const float*)table, w, w_dt, out, D, V, scale, eps,
+                       status);
+    else
+        return gfb_fail("gfb_embed_normed: unknown table type %d", table_dt);
+    return gfb_check(e, "gfb_embed_normed");
+}

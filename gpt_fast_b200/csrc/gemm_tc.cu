@@ -30,7 +30,7 @@
 
 GFB_DEFINE_LAST_ERROR()
 
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3, EPI_GELU = 4, EPI_RELU2 = 7, EPI_GLU_CLAMP = 8 };   // GELU: store gelu(acc), the exact (erf) form, as bfloat16; RELU2: store max(acc, 0)^2; GLU_CLAMP: see Groups
+enum { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3, EPI_GELU = 4, EPI_GELU_TANH = 5, EPI_RELU2 = 7, EPI_GLU_CLAMP = 8 };   // GELU: store gelu(acc), the exact (erf) form, as bfloat16; GELU_TANH: its tanh form; RELU2: store max(acc, 0)^2; GLU_CLAMP: see Groups
 
 // A product whose row tiles use different weight matrices (a mixture of experts with its rows sorted by expert): row tile i
 // multiplies with the rows [tile_group[i] * group_rows, + N) of the weight matrix; a tile whose entry is negative has no rows.
@@ -47,6 +47,8 @@ struct Groups {
 template <int EPI>
 __device__ __forceinline__ float fin(float x) {
     if (EPI == EPI_GELU) return 0.5f * x * (1.0f + erff(x * 0.70710678118654752440f));
+    if (EPI == EPI_GELU_TANH)           // 0.5 x (1 + tanh(z)) = x / (1 + e^(-2z)), z = sqrt(2 / pi) (x + 0.044715 x^3)
+        return __fdividef(x, 1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
     if (EPI == EPI_RELU2) { const float r = fmaxf(x, 0.f); return r * r; }
     return x;
 }
@@ -1250,6 +1252,7 @@ int dispatch_epi(int epi, int out_dt, const CUtensorMap& mx, const CUtensorMap& 
     if (epi == EPI_ADD) GO(EPI_ADD, float);
     if (epi == EPI_SWIGLU) GO(EPI_SWIGLU, bf16);
     if (epi == EPI_GELU && out_dt == GFB_BF16) GO(EPI_GELU, bf16);
+    if (epi == EPI_GELU_TANH && out_dt == GFB_BF16) GO(EPI_GELU_TANH, bf16);
     if (epi == EPI_RELU2 && out_dt == GFB_BF16) GO(EPI_RELU2, bf16);
     if (epi == EPI_STORE && out_dt == GFB_F32) GO(EPI_STORE, float);
     if (epi == EPI_STORE && out_dt == GFB_BF16) GO(EPI_STORE, bf16);
@@ -1272,7 +1275,7 @@ GFB_API int gfb_gemm_tc(const void* A, const void* W, void* out, int out_dt, int
     if (K <= 0 || K % 8) return gfb_fail("gfb_gemm_tc: K = %d must be a positive multiple of 8 (16-byte rows for TMA)", K);
     if (N % 8) return gfb_fail("gfb_gemm_tc: N = %d must be a multiple of 8", N);
     if (epi == EPI_SWIGLU && N % 16) return gfb_fail("gfb_gemm_tc: SwiGLU needs N %% 16 == 0, got %d", N);
-    if ((epi == EPI_GELU || epi == EPI_RELU2) && out_dt != GFB_BF16) return gfb_fail("gfb_gemm_tc: the GELU and squared-ReLU epilogues store bfloat16");
+    if ((epi == EPI_GELU || epi == EPI_GELU_TANH || epi == EPI_RELU2) && out_dt != GFB_BF16) return gfb_fail("gfb_gemm_tc: the GELU and squared-ReLU epilogues store bfloat16");
     if (((uintptr_t)A | (uintptr_t)W | (uintptr_t)out) & 15) return gfb_fail("gfb_gemm_tc: operands must be 16-byte aligned");
     if (stages < 2 || stages > MAX_STAGES) return gfb_fail("gfb_gemm_tc: stages = %d out of range", stages);
     if (bn < 512 && smem_bytes(bn, stages) > 227 * 1024) return gfb_fail("gfb_gemm_tc: %d stages of a %d-column tile exceed shared memory", stages, bn);
@@ -1310,6 +1313,7 @@ GFB_API int gfb_gemm_tc(const void* A, const void* W, void* out, int out_dt, int
         if (epi == EPI_ADD) return launch_pair<EPI_ADD, float>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
         if (epi == EPI_SWIGLU) return launch_pair<EPI_SWIGLU, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
         if (epi == EPI_GELU) return launch_pair<EPI_GELU, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
+        if (epi == EPI_GELU_TANH) return launch_pair<EPI_GELU_TANH, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
         if (epi == EPI_RELU2) return launch_pair<EPI_RELU2, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
         if (out_dt == GFB_F32) return launch_pair<EPI_STORE, float>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
         return launch_pair<EPI_STORE, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count2, status, stream);
@@ -1330,6 +1334,7 @@ GFB_API int gfb_gemm_tc(const void* A, const void* W, void* out, int out_dt, int
         if (epi == EPI_ADD) return launch_persistent<EPI_ADD, float>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
         if (epi == EPI_SWIGLU) return launch_persistent<EPI_SWIGLU, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
         if (epi == EPI_GELU) return launch_persistent<EPI_GELU, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
+        if (epi == EPI_GELU_TANH) return launch_persistent<EPI_GELU_TANH, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
         if (epi == EPI_RELU2) return launch_persistent<EPI_RELU2, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
         if (out_dt == GFB_F32) return launch_persistent<EPI_STORE, float>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
         return launch_persistent<EPI_STORE, bf16>(mx, my2, out, M, N, K, ldo, st, sm_count, status, stream);
@@ -1353,6 +1358,7 @@ GFB_API int gfb_gemm_tc(const void* A, const void* W, void* out, int out_dt, int
         if (epi == EPI_ADD) RED(EPI_ADD, float);
         else if (epi == EPI_SWIGLU) RED(EPI_SWIGLU, bf16);
         else if (epi == EPI_GELU) RED(EPI_GELU, bf16);
+        else if (epi == EPI_GELU_TANH) RED(EPI_GELU_TANH, bf16);
         else if (epi == EPI_RELU2) RED(EPI_RELU2, bf16);
         else if (out_dt == GFB_F32) RED(EPI_STORE, float);
         else RED(EPI_STORE, bf16);

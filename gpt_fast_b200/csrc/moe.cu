@@ -6,7 +6,9 @@
 //                       the `top` largest logits themselves, weighted by the softmax over just those, times scale.  Or (mode
 //                       ROUTE_SOFTMAX) s = softmax over all E logits, chosen by s + correction, weighted by s * scale.  With
 //                       `groups` > 1 only experts of the `keep` groups (of equal size, neighbours) whose largest choice
-//                       scores are largest can be chosen.  `shared` = 1: every token also runs expert number E with weight 1
+//                       scores are largest can be chosen (`group_terms` = 2: the groups whose two largest choice scores have the
+//                       largest sum).  Mode ROUTE_SIGMOID_PLAIN: weights s * scale, not divided by their sum.
+//                       `shared` = 1: every token also runs expert number E with weight 1
 // gfb_moe_glu           act[pair, f] = g * sigmoid(alpha g) * (u + shift),  g = min(gate_f . h, limit),
 //                       u = clamp(up_f . h, -limit, limit), for every (token, chosen expert) pair
 //                       or, for experts of two products (kind RELU2), act[pair, f] = max(up_f . h, 0)^2
@@ -36,13 +38,13 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf
 // ------------------------------------------------------------------------------------ router ----
 constexpr int MAX_EPL = 16;           // experts per lane: E <= 512
 constexpr int ROUTE_WARPS = 4;
-enum { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX = 2 };
+enum { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX = 2, ROUTE_SIGMOID_PLAIN = 3 };
 constexpr int MAX_GROUPS = 32;        // a lane keeps a group's score
 
 struct RouteArgs {
     int E, top;
     float scale;
-    int mode, groups, keep, shared;
+    int mode, groups, keep, group_terms, shared;
 };
 
 // one token's choice by one warp: `logits` are the token's E router logits
@@ -71,7 +73,8 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
         }
     }
     if (ra.groups > 1) {
-        // lane g keeps the largest choice score of group g; the `keep` best groups stay (the lowest index on ties)
+        // lane g keeps the score of group g, its largest choice score or the sum of its two largest; the `keep` best groups stay
+        // (the lowest index on ties)
         const int per = E / ra.groups;
         float score = -INFINITY;
         for (int g = 0; g < ra.groups; g++) {
@@ -79,7 +82,22 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
 #pragma unroll
             for (int i = 0; i < MAX_EPL; i++)
                 if ((lane + 32 * i) / per == g) m = fmaxf(m, c[i]);            // (experts beyond E are -inf)
-            m = gfb_warp_max(m);
+            const float top1 = gfb_warp_max(m);
+            if (ra.group_terms > 1 && per > 1) {
+                // the second largest: the first holder of the largest (by lane) looks at its other experts, every other lane at all
+                const int holder = __ffs(__ballot_sync(0xffffffffu, m == top1)) - 1;
+                float second = -INFINITY;
+                bool skip = lane == holder;
+#pragma unroll
+                for (int i = 0; i < MAX_EPL; i++)
+                    if ((lane + 32 * i) / per == g) {
+                        if (skip && c[i] == top1) skip = false;
+                        else second = fmaxf(second, c[i]);
+                    }
+                m = top1 + gfb_warp_max(second);
+            } else {
+                m = top1;
+            }
             if (lane == g) score = m;
         }
         unsigned kept = 0u;
@@ -127,7 +145,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
     }
     if (lane < top) {
         idx[lane] = mine_e;
-        weights[lane] = mode == ROUTE_SOFTMAX ? mine * scale : mode == ROUTE_SOFTMAX_TOP ? mine / sum * scale : mine / (sum + 1e-20f) * scale;
+        weights[lane] = mode == ROUTE_SOFTMAX || mode == ROUTE_SIGMOID_PLAIN ? mine * scale : mode == ROUTE_SOFTMAX_TOP ? mine / sum * scale : mine / (sum + 1e-20f) * scale;
     }
     if (ra.shared && lane == 0) {
         idx[top] = E;
@@ -140,6 +158,7 @@ static int check_route(const RouteArgs& ra, const char* what) {
     if (ra.top < 1 || ra.top > 32 || ra.top > ra.E) return gfb_fail("%s: %d of %d experts per token (1 to 32)", what, ra.top, ra.E);
     if (ra.groups < 1 || ra.groups > MAX_GROUPS || ra.E % ra.groups || ra.keep < 1 || ra.keep > ra.groups || ra.top > ra.keep * (ra.E / ra.groups))
         return gfb_fail("%s: %d experts from %d of %d groups of %d experts in all", what, ra.top, ra.keep, ra.groups, ra.E);
+    if (ra.group_terms < 1 || ra.group_terms > 2) return gfb_fail("%s: a group's score from %d choice scores (1 or 2)", what, ra.group_terms);
     return 0;
 }
 
@@ -157,9 +176,9 @@ moe_route_kernel(const float* __restrict__ logits, int ld, const void* __restric
 
 // idx int32 and weights float32 [T, top + shared]
 GFB_API int gfb_moe_route(const float* logits, int ld, const void* correction, int c_dt, int E, int top, float scale, int* idx,
-                          float* weights, int T, int mode, int groups, int keep, int shared, cudaStream_t stream) {
+                          float* weights, int T, int mode, int groups, int keep, int group_terms, int shared, cudaStream_t stream) {
     if (T <= 0) return 0;
-    const RouteArgs ra{E, top, scale, mode, groups, keep, shared ? 1 : 0};
+    const RouteArgs ra{E, top, scale, mode, groups, keep, group_terms, shared ? 1 : 0};
     if (check_route(ra, "gfb_moe_route")) return 1;
     cudaError_t e = gfb_launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(32 * ROUTE_WARPS), 0, stream, logits, ld,
                                correction, c_dt, ra, idx, weights, T);
@@ -227,10 +246,10 @@ moe_router_kernel(const T* __restrict__ h, const T* __restrict__ router, const v
 // h [T, D] and router [>= E + n_extra, D] of type dt (further rows are padding); few tokens only: a block per token.
 // The logits of the n_extra rows behind the experts' go to extra float32 [T, n_extra].
 GFB_API int gfb_moe_router(const void* h, const void* router, int dt, const void* correction, int c_dt, int E, int top, float scale,
-                           int* idx, float* weights, int T, int D, int mode, int groups, int keep, int shared, int n_extra, float* extra,
+                           int* idx, float* weights, int T, int D, int mode, int groups, int keep, int group_terms, int shared, int n_extra, float* extra,
                              cudaStream_t stream) {
     if (T <= 0) return 0;
-    const RouteArgs ra{E, top, scale, mode, groups, keep, shared ? 1 : 0};
+    const RouteArgs ra{E, top, scale, mode, groups, keep, group_terms, shared ? 1 : 0};
     if (check_route(ra, "gfb_moe_router")) return 1;
     if (n_extra < 0 || (n_extra > 0 && extra == nullptr)) return gfb_fail("gfb_moe_router: %d further rows without a place for their logits", n_extra);
     const size_t smem = (size_t)(D + E + n_extra) * sizeof(float);

@@ -13,7 +13,9 @@
 // of it (NORM_LAST).  `maps` > 1: every query head and every key head is `maps` vectors of dk side by side
 // (several score maps over one set of values); each is normed and rotated as a head of its own, and a cached
 // key row holds the `maps` vectors of its head one after the other.
-// One warp per (token, head); the head sits in shared memory between the steps.
+// A projection's biases (one number per column of the source row) are added ahead of everything else.
+// One warp per (token, head), the head in shared memory between the steps; with a norm over the whole projection one
+// block per token, the token's q, k and v in shared memory between the steps, so every number is read once.
 #include "common.cuh"
 
 GFB_DEFINE_LAST_ERROR()
@@ -28,8 +30,8 @@ __device__ __forceinline__ float ld_w(const void* p, int dt, int i) {
 template <typename T>
 __global__ void __launch_bounds__(WARPS * 32)
 qkv_prepare_kernel(const void* __restrict__ src, int S, size_t slice, int width, int q_off, int k_off, int v_off,
-                   T* __restrict__ q_out, GfbPagedKV kv, GfbBatch b, const float* __restrict__ table, int table_len,
-                   int rot_dims, int pairing, const void* q_norm, const void* k_norm, int w_dt, float eps, float k_scale,
+                   const void* __restrict__ bias, int b_dt, T* __restrict__ q_out, GfbPagedKV kv, GfbBatch b,
+                   const float* __restrict__ table, int table_len, int rot_dims, int pairing, const void* q_norm, const void* k_norm, int w_dt, float eps, float k_scale,
                    int H, int GK, int G, int maps, int dk, int dv, int dmax, int append, int norm_opts, int* status) {
     extern __shared__ float heads[];
     gfb_pdl_launch();
@@ -65,7 +67,8 @@ qkv_prepare_kernel(const void* __restrict__ src, int S, size_t slice, int width,
         if (is_q) for (int i = lane; i < dk; i += 32) dst[i] = gfb_from_f32<T>(0.f);     // q stays defined
         return;
     }
-    const size_t e0 = (size_t)t * width + (is_q ? q_off + head * dk : is_k ? k_off + (head - H) * dk : v_off + (head - H - GK) * dv);
+    const int c0 = is_q ? q_off + head * dk : is_k ? k_off + (head - H) * dk : v_off + (head - H - GK) * dv;
+    const size_t e0 = (size_t)t * width + c0;
     float ss = 0.f;
     for (int i = lane; i < d; i += 32) {
         float x;
@@ -76,6 +79,7 @@ qkv_prepare_kernel(const void* __restrict__ src, int S, size_t slice, int width,
         } else {
             x = gfb_to_f32(((const T*)src)[e0 + i]);
         }
+        if (bias != nullptr) x += ld_w(bias, b_dt, c0 + i);
         v[i] = x;
         ss += x * x;
     }
@@ -94,6 +98,7 @@ qkv_prepare_kernel(const void* __restrict__ src, int S, size_t slice, int width,
             } else {
                 x = gfb_to_f32(((const T*)src)[p0 + i]);
             }
+            if (bias != nullptr) x += ld_w(bias, b_dt, (is_q ? q_off : k_off) + i);
             tot += x * x;
         }
         tot = gfb_warp_sum(tot);
@@ -127,14 +132,147 @@ qkv_prepare_kernel(const void* __restrict__ src, int S, size_t slice, int width,
     for (int i = lane; i < d; i += 32) dst[i] = gfb_from_f32<T>(v[i] * f);
 }
 
+// ---- a norm over the whole projection: a block per token -----------------------------------------------
+// Shared memory holds the token's q (H heads of dk), k (G of dk) and v (G of dv), biases added.  N = 4: everything moves four
+// numbers at a time (columns, head sizes and offsets are multiples of four); N = 1: any sizes.
+template <typename T, int N> struct alignas(N * sizeof(T)) AlignedPack { T v[N]; };
+
+template <typename T, int N>
+__device__ __forceinline__ float stage_columns(float* dst, const void* __restrict__ src, int S, size_t slice, size_t row, int c0, int n,
+                                               const void* __restrict__ bias, int b_dt) {
+    float ss = 0.f;
+    for (int i = threadIdx.x * N; i < n; i += blockDim.x * N) {
+        float x[N];
+        if (S > 0) {
+            const float* p = (const float*)src + row + c0 + i;
+#pragma unroll
+            for (int e = 0; e < N; e++) x[e] = 0.f;
+            constexpr int W = 4;                                   // partial sums in flight together, added in ascending order
+            for (int k = 0; k < S; k += W) {
+                AlignedPack<float, N> a[W];
+#pragma unroll
+                for (int u = 0; u < W; u++) a[u] = *reinterpret_cast<const AlignedPack<float, N>*>(p + (size_t)min(k + u, S - 1) * slice);
+#pragma unroll
+                for (int u = 0; u < W; u++)
+                    if (k + u < S) {
+#pragma unroll
+                        for (int e = 0; e < N; e++) x[e] += a[u].v[e];
+                    }
+            }
+        } else {
+            const AlignedPack<T, N> a = *reinterpret_cast<const AlignedPack<T, N>*>((const T*)src + row + c0 + i);
+#pragma unroll
+            for (int e = 0; e < N; e++) x[e] = gfb_to_f32(a.v[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < N; e++) {
+            if (bias != nullptr) x[e] += ld_w(bias, b_dt, c0 + i + e);
+            dst[i + e] = x[e];
+            ss += x[e] * x[e];
+        }
+    }
+    return ss;
+}
+
+// numbers i .. i + N - 1 of a normed head (v: the head as projected, w0: its first weight), rotated where they lie in the first rot_dims
+template <typename T, int N>
+__device__ __forceinline__ AlignedPack<T, N> finish_columns(const float* v, int i, float r, const void* w, int w_dt, int w0, const float* cs, int rot_dims,
+                                                            int pairing, float f) {
+    AlignedPack<T, N> o;
+    const int half = rot_dims >> 1;
+#pragma unroll
+    for (int e = 0; e < N; e++) {
+        const int j = i + e;
+        float x = v[j] * r * (w != nullptr ? ld_w(w, w_dt, w0 + j) : 1.f);
+        if (j < rot_dims) {
+            const int pair = pairing == 1 ? (j < half ? j : j - half) : j >> 1;
+            const bool first = pairing == 1 ? j < half : !(j & 1);
+            const int other = pairing == 1 ? (first ? j + half : j - half) : j ^ 1;
+            const float y = v[other] * r * (w != nullptr ? ld_w(w, w_dt, w0 + other) : 1.f);
+            const float c = cs[2 * pair], sn = cs[2 * pair + 1];
+            x = first ? x * c - y * sn : x * c + y * sn;
+        }
+        o.v[e] = gfb_from_f32<T>(x * f);
+    }
+    return o;
+}
+
+template <typename T, int N>
+__global__ void qkv_prepare_token_kernel(const void* __restrict__ src, int S, size_t slice, int width, int q_off, int k_off, int v_off,
+                                         const void* __restrict__ bias, int b_dt, T* __restrict__ q_out, GfbPagedKV kv, GfbBatch b,
+                                         const float* __restrict__ table, int table_len, int rot_dims, int pairing, const void* q_norm,
+                                         const void* k_norm, int w_dt, float eps, float k_scale, int H, int G, int dk, int dv, int append,
+                                         int* status) {
+    extern __shared__ __align__(16) float heads[];
+    __shared__ float scratch[32];
+    gfb_pdl_launch();
+    gfb_pdl_wait();
+    const int t = blockIdx.x;
+    const int s = b.tok_seq[t];
+    const int slot = b.slots[s];
+    const int pos = b.lengths[slot] + (t - b.cu_seqlens[s]);
+    const int nq = H * dk, nk = append ? G * dk : 0, nv = append ? G * dv : 0;
+    bool ok = pos >= 0 && (table == nullptr || pos < table_len);
+    int page = -1, off = 0;
+    if (append && ok) {
+        const int pi = pos / kv.page_size;
+        off = pos - pi * kv.page_size;
+        page = pi < kv.max_pages ? kv.page_table[(size_t)slot * kv.max_pages + pi] : -1;
+        ok = page >= 0 && page < kv.n_pages;
+    }
+    if (!ok) {
+        if (threadIdx.x == 0) gfb_report(status, GFB_ERR_CACHE_RANGE, t, pos);
+        for (int i = threadIdx.x; i < nq; i += blockDim.x) q_out[(size_t)t * nq + i] = gfb_from_f32<T>(0.f);     // q stays defined
+        return;
+    }
+    const size_t row = (size_t)t * width;
+    float* ks = heads + nq;
+    float* vs = ks + nk;
+    float sq = stage_columns<T, N>(heads, src, S, slice, row, q_off, nq, bias, b_dt);
+    float sk = stage_columns<T, N>(ks, src, S, slice, row, k_off, nk, bias, b_dt);
+    stage_columns<T, N>(vs, src, S, slice, row, v_off, nv, bias, b_dt);
+    sq = gfb_block_sum(sq, scratch);                               // (these also order the staged numbers)
+    sk = gfb_block_sum(sk, scratch);
+    __syncthreads();
+    const float rq = q_norm != nullptr ? 1.0f / sqrtf(sq / (float)nq + eps) : 1.f;
+    const float rk = k_norm != nullptr ? 1.0f / sqrtf(sk / (float)max(nk, 1) + eps) : 1.f;
+    const float* cs = table != nullptr ? table + (size_t)pos * rot_dims : nullptr;
+    for (int i = threadIdx.x * N; i < nq; i += blockDim.x * N) {
+        const int h = i / dk, j = i - h * dk;
+        *reinterpret_cast<AlignedPack<T, N>*>(q_out + (size_t)t * nq + i) =
+            finish_columns<T, N>(heads + h * dk, j, rq, q_norm, w_dt, h * dk, cs, rot_dims, pairing, 1.f);
+    }
+    for (int i = threadIdx.x * N; i < nk; i += blockDim.x * N) {
+        const int g = i / dk, j = i - g * dk;
+        T* dst = (T*)kv.k_pool + (((size_t)page * G + g) * kv.page_size + off) * dk + j;
+        *reinterpret_cast<AlignedPack<T, N>*>(dst) = finish_columns<T, N>(ks + g * dk, j, rk, k_norm, w_dt, g * dk, cs, rot_dims, pairing, k_scale);
+    }
+    for (int i = threadIdx.x * N; i < nv; i += blockDim.x * N) {
+        const int g = i / dv, j = i - g * dv;
+        AlignedPack<T, N> o;
+#pragma unroll
+        for (int e = 0; e < N; e++) o.v[e] = gfb_from_f32<T>(vs[i + e]);
+        *reinterpret_cast<AlignedPack<T, N>*>((T*)kv.v_pool + (((size_t)page * G + g) * kv.page_size + off) * dv + j) = o;
+    }
+}
+
+template <typename T, int N, typename... A>
+static cudaError_t launch_token(size_t smem, int n_tokens, int threads, cudaStream_t stream, A... args) {
+    if (smem > 40 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(qkv_prepare_token_kernel<T, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+    }
+    return gfb_launch(qkv_prepare_token_kernel<T, N>, dim3((unsigned)n_tokens), dim3((unsigned)threads), smem, stream, args...);
+}
+
 // src: [T, width] of type dt, or with n_partials > 0 float32 [n_partials][T][width]; q at q_off (H heads of dk), k at
-// k_off (G heads of dk), v at v_off (G heads of dv).  table (or null: no rotation): float32 [table_len][rot_dims/2][2].
+// k_off (G heads of dk), v at v_off (G heads of dv).  bias (or null): [width] of type b_dt.  table (or null: no rotation): float32 [table_len][rot_dims/2][2].
 // q_norm / k_norm (or null): [dk] of type w_dt, or with NORM_WHOLE [H * dk] and [G * dk].  append = 0: only q is produced.
 // norm_opts: NORM_WHOLE | NORM_BARE (a per-head norm also where no weight is given) | NORM_LAST (the per-head norm follows
 // the rotation) | Q_SPREAD (q_out is [T, H * maps, maps * dk], zeroed by the caller; query j is written at columns
 // (j mod maps) * dk of row j).  maps >= 1: H and G count heads; q_out is [T, H * maps, dk], key rows of the cache hold maps * dk numbers.
-GFB_API int gfb_qkv_prepare(const void* src, int n_partials, int width, int q_off, int k_off, int v_off, void* q_out, int dt,
-                            void* k_pool, void* v_pool, const int* page_table, int max_pages, int page_size, int n_pages,
+GFB_API int gfb_qkv_prepare(const void* src, int n_partials, int width, int q_off, int k_off, int v_off, const void* bias, int b_dt,
+                            void* q_out, int dt, void* k_pool, void* v_pool, const int* page_table, int max_pages, int page_size, int n_pages,
                             const int* cu_seqlens, const int* tok_seq, const int* slots, const int* lengths, int n_seqs,
                             int n_tokens, const float* table, int table_len, int rot_dims, int pairing,
                             const void* q_norm, const void* k_norm, int w_dt, float eps, float k_scale,
@@ -154,8 +292,23 @@ GFB_API int gfb_qkv_prepare(const void* src, int n_partials, int width, int q_of
     if (smem > 48 * 1024) return gfb_fail("gfb_qkv_prepare: heads of %d exceed the kernel's shared memory", dmax);
     const size_t slice = (size_t)n_tokens * width;
     cudaError_t e;
+    const size_t token_smem = ((size_t)H * dk + (append ? (size_t)G * (dk + dv) : 0)) * sizeof(float);
+    if ((norm_opts & NORM_WHOLE) && maps == 1 && !(norm_opts & ~NORM_WHOLE) && token_smem <= 160 * 1024) {
+        const bool four = ((q_off | k_off | v_off | width | dk | dv) & 3) == 0
+                          && (((uintptr_t)src | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) == 0;
+        const long cols = (long)H * dk + (append ? (long)G * (dk + dv) : 0);
+        const int threads = cols <= 1024 ? 128 : n_tokens <= 128 && cols > 2048 ? 512 : 256;
+#define TOKEN(T, N) e = launch_token<T, N>(token_smem, n_tokens, threads, stream, src, n_partials, slice, width, q_off, k_off, v_off, bias, b_dt, \
+                                           (T*)q_out, kv, b, table, table_len, table != nullptr ? rot_dims : 0, pairing, q_norm, k_norm, w_dt, eps, k_scale, H, G, \
+                                           dk, dv, append, status)
+        if (dt == GFB_BF16) { if (four) TOKEN(__nv_bfloat16, 4); else TOKEN(__nv_bfloat16, 1); }
+        else if (dt == GFB_F32) { if (four) TOKEN(float, 4); else TOKEN(float, 1); }
+        else return gfb_fail("gfb_qkv_prepare: unknown type %d", dt);
+#undef TOKEN
+        return gfb_check(e, "gfb_qkv_prepare (token)");
+    }
 #define GO(T) e = gfb_launch(qkv_prepare_kernel<T>, dim3((unsigned)blocks), dim3(WARPS * 32), smem, stream, src, n_partials, slice, \
-                             width, q_off, k_off, v_off, (T*)q_out, kv, b, table, table_len, rot_dims, pairing, q_norm, k_norm, \
+                             width, q_off, k_off, v_off, bias, b_dt, (T*)q_out, kv, b, table, table_len, rot_dims, pairing, q_norm, k_norm, \
                              w_dt, eps, k_scale, HQ, GK, G, maps, dk, dv, dmax, append, norm_opts, status)
     if (dt == GFB_BF16) GO(__nv_bfloat16);
     else if (dt == GFB_F32) GO(float);

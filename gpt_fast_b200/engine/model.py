@@ -16,6 +16,7 @@ from ..cache import Cache, CacheNeeds, EntryView
 from ..config.spec import ModelSpec, PartSpec
 from ..ops.types import BatchMeta
 from ..parts.residual import Residual
+from ..parts.streams import Streams
 from ..parts import EMBEDDINGS, JUNCTIONS, NORMS, POSITIONS, build_block, build_part
 from ..weights.loader import ParamSpec
 
@@ -56,13 +57,15 @@ class Transformer:
 
         self.blocks = [build_block(ls, spec.dim, self.dtype, position_for(ls.position)) for ls in spec.layers]
         self.positions = [obj for _, obj in positions]
+        if any(getattr(b, "takes_streams", False) != bool(spec.streams) for b in self.blocks):
+            raise ValueError("a model with several residual streams is made of blocks that take streams, any other model of blocks that do not")
         self.final_norm = build_part(NORMS, spec.final_norm, dtype=self.dtype)
         self.embedding = None if spec.embedding is None else build_part(EMBEDDINGS, spec.embedding, dtype=self.dtype)
         self.junctions = [build_part(JUNCTIONS, ps, dtype=self.dtype) for ps in spec.junctions]
         self.embed_weight = None
         self.head_weight = None
         self.token_table = None            # [vocab, spec.token_table]: what token inputs read of a token
-        self.after_layer = None            # a callable(Residual) run behind every layer of a step (tests look at the stream)
+        self.after_layer = None            # a callable(stream) run behind every layer of a step (tests look at the stream)
 
     # ---- parameters -------------------------------------------------------------
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -225,7 +228,7 @@ class Transformer:
         x0 = x                                  # the embedding output, which junctions read again
         if self.junctions and self.spec.schedule[0].junction is None:
             x = x0.clone()                      # layers ahead of the first junction write into the stream
-        x = Residual(x)
+        x = Streams(x, self.spec.streams) if self.spec.streams else Residual(x)
         for e in self.spec.schedule:
             if e.junction is not None:
                 self.junctions[e.junction].forward(x, x0, e.turn)
@@ -241,7 +244,7 @@ class Transformer:
         logits = torch.empty(W, self.vocab_size, dtype=torch.float32, device=self.device)
         if W:
             h = torch.empty(W, self.dim, dtype=self.dtype, device=self.device)
-            self.final_norm.forward(x, h, want_rows)
+            self.final_norm.forward(x.total() if self.spec.streams else x, h, want_rows)
             ops.linear(h, self.head_weight, logits)
             if self.spec.logit_cap is not None:
                 ops.softcap(logits, float(self.spec.logit_cap))

@@ -106,6 +106,12 @@ def embed_positions(tokens, table, positions, out, batch: BatchMeta, scale: floa
     return kernels().embed_positions(tokens, table, positions, out, batch, scale)
 
 
+def embed_normed(tokens, table, weight, eps: float, out, status, scale: float = 1.0):
+    """out[t] = e / sqrt(mean(e^2) + eps) * weight with e = table[tokens[t]] * scale, in 32-bit.  weight [D] (bfloat16 or float32);
+    out float32 [T, D]."""
+    return kernels().embed_normed(tokens, table, weight, eps, out, status, scale)
+
+
 def embed_hashed(tokens, table, extra, out, batch: BatchMeta, prev, buckets: int, mul_prev: int, mul_cur: int, scale: float = 1.0):
     """out[t] = table[tokens[t]] * scale + extra[(previous token * mul_prev + tokens[t] * mul_cur) mod buckets], with
     extra's row `buckets` for a sequence's first token.  extra [buckets + 1, D]; prev int32 [n_slots] is per-sequence
@@ -144,6 +150,18 @@ def layernorm_multi(x, branches=(), outs=(), rows=None, rms: bool = False):
     eps) * weight in the compute type; weight None (one output only): the new row itself.  rows int32 [R] gathers input rows (not together with branches).  rms=True:
     the root-mean-square form (no mean)."""
     return kernels().layernorm_multi(x, branches, outs, rows, rms)
+
+
+def streams(x, n: int, shared: bool = False, x_out=None, mix=None, leave=None, branches=(), enter=None, weight=None, eps: float = 0.0,
+            out=None, rows=None):
+    """Several residual streams per token: one sublayer's output on its way into them and the next one's input on its way out.
+    x float32 [n, T, D] (or, `shared`, [T, D]: all n streams are this tensor).  With mix (float32 [n, n], indexed from, to) and
+    leave (float32 [n]): x_t <- sum_s mix[s, t] x_s + leave[t] * y, all streams at once, y the sum of `branches` (up to two, each a
+    float32 [T, D] tensor or partial sums [S, T, D] added in ascending order), written to x_out [n, T, D] (x itself where it is not
+    shared; None: not written).  Then u = sum_t enter[t] x_t (enter float32 [n]; None: ones) and out [R, D] = u / sqrt(mean(u^2) +
+    eps) * weight, or u itself without a weight; out None: nothing.  rows int32 [R]: the rows of x that `out` is made of (x_out must
+    be None then)."""
+    return kernels().streams(x, n, shared, x_out, mix, leave, branches, enter, weight, eps, out, rows)
 
 
 def latent_prepare(src, q_off: int, kv_off: int, q_out, kv: PagedKV, batch: BatchMeta, n_head: int, head_dim: int,
@@ -255,7 +273,7 @@ def gated_norm(y, gate, gate_off: int, weight, out, group: int, eps: float, act:
 def qkv_prepare(src, partials, offsets, q_out, kv: PagedKV, batch: BatchMeta, n_head: int, n_kv: int, head_dim: int,
                 v_head_dim: int, table=None, rot_dims: int = 0, pairing: str = "half", q_norm=None, k_norm=None,
                 norm_eps: float = 0.0, k_scale: float = 1.0, append: bool = True, norm_whole: bool = False,
-                norm_bare: bool = False, norm_last: bool = False, maps: int = 1, q_spread: bool = False):
+                norm_bare: bool = False, norm_last: bool = False, maps: int = 1, q_spread: bool = False, bias=None):
     """From a projection's row to attention's inputs.  src [T, W] holds q (H heads of head_dim), k (G heads of
     head_dim) and v (G heads of v_head_dim) at the column offsets `offsets` = (q, k, v); with `partials` (float32
     [S, T, W]) src is their sum.  Per head, in this order: root-mean-square norm of q and k with the weights
@@ -266,7 +284,12 @@ def qkv_prepare(src, partials, offsets, q_out, kv: PagedKV, batch: BatchMeta, n_
     without a weight.  norm_last: the per-head norm follows the rotation.  maps > 1: every query head and every key head
     is `maps` vectors of head_dim side by side, each normed and rotated like a head; q_out is [T, H * maps, head_dim]
     and a cached key row holds maps * head_dim numbers.  q_spread (see `spread_queries`): q_out is [T, H * maps,
-    maps * head_dim], zeroed by the caller, and query j goes to columns (j mod maps) * head_dim of its row."""
+    maps * head_dim], zeroed by the caller, and query j goes to columns (j mod maps) * head_dim of its row.  bias [W] (bfloat16 or float32): added to the row ahead
+    of everything else."""
+    if bias is not None:
+        return kernels().qkv_prepare(src, partials, offsets, q_out, kv, batch, n_head, n_kv, head_dim, v_head_dim, table,
+                                     rot_dims, pairing, q_norm, k_norm, norm_eps, k_scale, append, norm_whole=norm_whole,
+                                     norm_bare=norm_bare, norm_last=norm_last, maps=maps, q_spread=q_spread, bias=bias)
     if q_spread:
         return kernels().qkv_prepare(src, partials, offsets, q_out, kv, batch, n_head, n_kv, head_dim, v_head_dim, table,
                                      rot_dims, pairing, q_norm, k_norm, norm_eps, k_scale, append, norm_whole=norm_whole,
@@ -317,8 +340,9 @@ def moe_route(logits, correction, top: int, scale: float, idx, weights, score: s
     the `top` experts with the largest s + correction (lowest index on ties) go to idx int32 [T, top], and
     weights float32 [T, top] = their s / (sum of the chosen s + 1e-20) * scale.  score 'softmax_top': the `top` largest
     logits (+ correction) are chosen and weights = softmax over the chosen logits * scale.  score 'softmax': s = softmax over
-    all E logits, weights = the chosen s * scale.  groups = (count, keep): the experts are `count` equal groups of neighbours
-    and only those of the `keep` groups with the largest single choice score can be chosen.  shared: idx and weights are
+    all E logits, weights = the chosen s * scale.  score 'sigmoid_plain': 'sigmoid' with weights = the chosen s * scale, not divided
+    by their sum.  groups = (count, keep[, terms]): the experts are `count` equal groups of neighbours and only those of the `keep`
+    best groups can be chosen; a group's score is its largest choice score (terms 1) or the sum of its two largest (2).  shared: idx and weights are
     [T, top + 1] and the last entry of every row is expert number E with weight 1."""
     kw = _route_options(score, groups, shared)
     return kernels().moe_route(logits, correction, top, scale, idx, weights, **kw)
@@ -327,7 +351,7 @@ def moe_route(logits, correction, top: int, scale: float, idx, weights, score: s
 def _route_options(score, groups, shared) -> dict:
     kw = {} if score == "sigmoid" else {"score": score}
     if groups is not None and tuple(groups)[0] > 1:
-        kw["groups"] = (int(groups[0]), int(groups[1]))
+        kw["groups"] = tuple(int(g) for g in groups)
     if shared:
         kw["shared"] = True
     return kw

@@ -12,7 +12,7 @@ from .types import BatchMeta, PagedKV
 _DT = {torch.float32: 0, torch.bfloat16: 1}
 _EPI = {"store": 0, "add": 1, "swiglu": 2, "gelu": 4, "gelu_tanh": 5, "silu": 6, "relu2": 7}
 _UNARY = ("gelu", "gelu_tanh", "silu", "relu2")
-_TC_UNARY = ("gelu", "relu2")             # the unary epilogues the tensor-core product has (they store bfloat16)
+_TC_UNARY = ("gelu", "gelu_tanh", "relu2")             # the unary epilogues the tensor-core product has (they store bfloat16)
 _PAIRING = {"interleaved": 0, "half": 1}
 
 
@@ -130,6 +130,56 @@ class CudaKernels:
         _need(out, torch.float32, (T, D), "embedding output")
         self._call("core", "gfb_embed", _ptr(tokens), _ptr(table), c_int(_dt(table)), _ptr(out),
                    c_int(T), c_int(D), c_int(V), c_float(scale), _ptr(status), _stream())
+
+    def embed_normed(self, tokens, table, weight, eps, out, status, scale=1.0):
+        T = tokens.shape[0]
+        V, D = table.shape
+        _need(tokens, torch.int32, (T,), "tokens")
+        _need(table, name="embedding table")
+        _need(weight, shape=(D,), name="embedding norm weight")
+        _need(out, torch.float32, (T, D), "embedding output")
+        self._call("embedding", "gfb_embed_normed", _ptr(tokens), _ptr(table), c_int(_dt(table)), _ptr(weight), c_int(_dt(weight)), _ptr(out),
+                   c_int(T), c_int(D), c_int(V), c_float(scale), c_float(eps), _ptr(status), _stream())
+
+    MAX_STREAMS = 16
+
+    def streams(self, x, n, shared=False, x_out=None, mix=None, leave=None, branches=(), enter=None, weight=None, eps=0.0, out=None,
+                rows=None):
+        T, D = x.shape[-2:]
+        _need(x, torch.float32, (T, D) if shared else (n, T, D), "streams")
+        if not 1 <= n <= self.MAX_STREAMS:
+            _fail(f"{n} streams (1 to {self.MAX_STREAMS})")
+        if (mix is None) != (leave is None) or (mix is None and (branches or x_out is not None)):
+            _fail("a sublayer's output goes into the streams with a mixing matrix and a factor per stream")
+        if len(branches) > 2:
+            _fail("at most two addends")
+        if mix is not None:
+            _need(mix, torch.float32, (n, n), "mixing matrix")
+            _need(leave, torch.float32, (n,), "factors of the output")
+        if enter is not None:
+            _need(enter, torch.float32, (n,), "factors of the input")
+        b_args = []
+        for y in list(branches) + [None] * (2 - len(branches)):
+            S = 0
+            if y is not None:
+                S = y.shape[0] if y.dim() == 3 else 0
+                _need(y, torch.float32, (S, T, D) if S else (T, D), "output of a sublayer")
+            b_args += [_ptr(y), c_int(S)]
+        R = T
+        if rows is not None:
+            if out is None or x_out is not None:
+                _fail("a gather of rows has an output and writes no streams")
+            R = out.shape[0]
+            _need(rows, torch.int32, (R,), "rows")
+        if x_out is not None:
+            _need(x_out, torch.float32, (n, T, D), "new streams")
+        if out is not None:
+            _need(out, shape=(R, D), name="norm output")
+        if weight is not None:
+            _need(weight, shape=(D,), name="norm weight")
+        self._call("streams", "gfb_streams", _ptr(x), c_long(0 if shared else T * D), _ptr(x_out), c_long(T * D), c_int(n), _ptr(mix), _ptr(leave),
+                   *b_args, c_long(T * D), _ptr(enter), _ptr(weight), c_int(_dt(weight) if weight is not None else 0), c_float(eps), _ptr(out),
+                   c_int(_dt(out) if out is not None else 0), _ptr(rows), c_int(R), c_int(D), _stream())
 
     def embed_hashed(self, tokens, table, extra, out, batch, prev, buckets, mul_prev, mul_cur, scale=1.0):
         T = tokens.shape[0]
@@ -514,7 +564,7 @@ class CudaKernels:
 
     def qkv_prepare(self, src, partials, offsets, q_out, kv, batch, n_head, n_kv, head_dim, v_head_dim, table=None, rot_dims=0,
                     pairing="half", q_norm=None, k_norm=None, norm_eps=0.0, k_scale=1.0, append=True, norm_whole=False,
-                    norm_bare=False, norm_last=False, maps=1, q_spread=False):
+                    norm_bare=False, norm_last=False, maps=1, q_spread=False, bias=None):
         T = batch.n_tokens
         if norm_whole and (norm_bare or norm_last or maps != 1):
             _fail("a norm over the whole projection has weights, runs ahead of the rotation and knows one map per head")
@@ -542,13 +592,15 @@ class CudaKernels:
                 w_dt = _dt(wn)
         if q_norm is not None and k_norm is not None and q_norm.dtype != k_norm.dtype:
             _fail("the q and k norm weights must have one type")
+        if bias is not None:
+            _need(bias, shape=(W,), name="bias of the projection")
         if append:
             _need(kv.k_pool, q_out.dtype, name="key pool")
             if tuple(kv.k_pool.shape[1:]) != (n_kv, kv.page_size, head_dim * maps) or tuple(kv.v_pool.shape[1:]) != (n_kv, kv.page_size, v_head_dim):
                 _fail(f"cache pages are {tuple(kv.k_pool.shape[1:])} / {tuple(kv.v_pool.shape[1:])}, the layer needs "
                       f"{(n_kv, kv.page_size, head_dim * maps)} / {(n_kv, kv.page_size, v_head_dim)}")
         self._call("qkv_prepare", "gfb_qkv_prepare", _ptr(source), c_int(n_part), c_int(W), c_int(q_off), c_int(k_off), c_int(v_off),
-                   _ptr(q_out), c_int(_dt(q_out)), *self._kv_args(kv), *self._batch_args(batch), _ptr(table),
+                   _ptr(bias), c_int(_dt(bias) if bias is not None else 0), _ptr(q_out), c_int(_dt(q_out)), *self._kv_args(kv), *self._batch_args(batch), _ptr(table),
                    c_int(table.shape[0] if table is not None else 0), c_int(rot_dims if table is not None else 0),
                    c_int(_PAIRING[pairing]), _ptr(q_norm), _ptr(k_norm), c_int(w_dt), c_float(norm_eps), c_float(k_scale),
                    c_int(n_head), c_int(n_kv), c_int(head_dim), c_int(v_head_dim), c_int(1 if append else 0),
@@ -611,13 +663,14 @@ class CudaKernels:
     MOE_PAIR_ROWS_PER_EXPERT = 384     # (token, expert) pairs per expert from which the row tiles have 256 rows
     _EPI_GLU_CLAMP = 8
 
-    _ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1, "softmax": 2}
+    _ROUTE_SCORES = {"sigmoid": 0, "softmax_top": 1, "softmax": 2, "sigmoid_plain": 3}
     MOE_MAX_GROUPS = 32
 
     def _route_args(self, score, groups, shared):
         if score not in self._ROUTE_SCORES:
             _fail(f"unknown router score '{score}'")
-        return (c_int(self._ROUTE_SCORES[score]), c_int(groups[0]), c_int(groups[1]), c_int(1 if shared else 0))
+        return (c_int(self._ROUTE_SCORES[score]), c_int(groups[0]), c_int(groups[1]), c_int(groups[2] if len(groups) > 2 else 1),
+                c_int(1 if shared else 0))
 
     def moe_route(self, logits, correction, top, scale, idx, weights, score="sigmoid", groups=(1, 1), shared=False):
         T, slots = logits.shape[0], top + (1 if shared else 0)

@@ -33,6 +33,8 @@ Options beyond gpt-fast's attention, each off by default:
   values_are_keys  no value projection: a position's values are its keys as projected, ahead of norm and rotation
   softcap          the scaled score s becomes softcap * tanh(s / softcap)
   keep_first       with a window: the sequence's first `keep_first` positions stay visible to every later query
+  bias             the q, k and v projections have biases (parameters bq, bk, bv), added ahead of everything else
+  sink_value       a sink that is a constant, the same for every head (0: one is added to the softmax denominator)
 With none of them the rotate-and-append kernel and the tensor-core attention kernels run; the others go through
 `ops.qkv_prepare` and the options of `ops.attention`."""
 import math
@@ -68,7 +70,8 @@ class Attention:
                  qk_norm_eps: Optional[float] = None, chunk: Optional[int] = None, sink: bool = False,
                  qk_norm_whole: bool = False, conv_taps: Optional[int] = None, distance_bias: Optional[dict] = None,
                  gate: Optional[str] = None, shared_kv: bool = False, qk_norm_weight: bool = True, qk_norm_last: bool = False,
-                 values_are_keys: bool = False, softcap: Optional[float] = None, keep_first: int = 0):
+                 values_are_keys: bool = False, softcap: Optional[float] = None, keep_first: int = 0, bias: bool = False,
+                 sink_value: Optional[float] = None):
         if n_head % n_kv:
             raise ValueError(f"{n_head} query heads do not divide into {n_kv} key/value heads")
         if chunk is not None and chunk < 1:
@@ -86,6 +89,11 @@ class Attention:
         self.values_are_keys = bool(values_are_keys)
         self.softcap = float(softcap) if softcap else None
         self.keep_first = int(keep_first or 0)
+        self.has_bias, self.sink_value = bool(bias), None if sink_value is None else float(sink_value)
+        if self.has_bias and (conv_taps or values_are_keys):
+            raise ValueError("biases of the projections do not go with a convolution behind them or with values that are the keys")
+        if self.has_sink and self.sink_value is not None:
+            raise ValueError("a sink is learned or constant, not both")
         if self.softcap is not None and not self.softcap > 0:
             raise ValueError(f"a soft cap of {softcap} on the scores")
         if self.keep_first < 0:
@@ -105,12 +113,12 @@ class Attention:
             elif kind != "slopes":
                 raise ValueError(f"a distance bias is of kind 'slopes' or 'table', not {kind!r}")
         extras = (self.qk_norm_whole or self.conv_taps or self.distance_bias is not None or gate is not None or self.shared_kv
-                  or self.values_are_keys or self.softcap is not None or self.keep_first)
+                  or self.values_are_keys or self.softcap is not None or self.keep_first or self.has_bias or self.sink_value is not None)
         self.plain = (position is not None and self.v_head_dim == head_dim and self.qk_norm_eps is None
                       and chunk is None and not self.has_sink and getattr(position, "head_dim", head_dim) == head_dim
                       and not extras)
         self.wqkv = self.wo = self.q_norm = self.k_norm = self.sink = None
-        self.conv = self.bias_table = self.slopes = None
+        self.conv = self.bias_table = self.slopes = self.qkv_bias = None
         # columns of the fused projection: q, then k and v (unless shared), then the gates
         self.kv_cols = 0 if self.shared_kv else n_kv * head_dim if self.values_are_keys else n_kv * (head_dim + self.v_head_dim)
         self.conv_channels = n_head * head_dim + self.kv_cols
@@ -127,6 +135,10 @@ class Attention:
             specs["q_norm"] = ParamSpec(((H if self.qk_norm_whole else 1) * d,), "vector")
             if not self.shared_kv:
                 specs["k_norm"] = ParamSpec(((G if self.qk_norm_whole else 1) * d,), "vector")
+        if self.has_bias:
+            specs["bq"] = ParamSpec((H * d,), "vector")
+            if not self.shared_kv:
+                specs.update(bk=ParamSpec((G * d,), "vector"), bv=ParamSpec((G * dv,), "vector"))
         if self.has_sink:
             specs["sink"] = ParamSpec((H,), "vector")
         if self.conv_taps:
@@ -145,7 +157,7 @@ class Attention:
         rows = [tensors["wq"]] + ([] if self.shared_kv else [tensors["wk"]] if self.values_are_keys else [tensors["wk"], tensors["wv"]])
         if self.gate is not None:
             rows.append(tensors["wg"])
-        self.wqkv = torch.cat(rows).contiguous() if self.plain or len(rows) == 3 and self.gate is None else _pad_rows(torch.cat(rows))
+        self.wqkv = torch.cat(rows).contiguous() if self.plain or len(rows) == 3 and self.gate is None and not self.has_bias else _pad_rows(torch.cat(rows))
         self.wo = tensors["wo"]
         if self.qk_norm_eps is not None and self.qk_norm_weight:
             self.q_norm = tensors["q_norm"]
@@ -153,6 +165,12 @@ class Attention:
         if self.has_sink:
             self._sink_stored = tensors["sink"]
             self.sink = tensors["sink"].float().contiguous()        # softmax terms are 32-bit
+        elif self.sink_value is not None:
+            self.sink = torch.full((self.n_head,), self.sink_value, dtype=torch.float32, device=self.wo.device)
+        if self.has_bias:
+            rows = [tensors["bq"]] + ([] if self.shared_kv else [tensors["bk"], tensors["bv"]])
+            total = torch.cat([r.float() for r in rows])
+            self.qkv_bias = torch.cat([total, total.new_zeros(self.wqkv.shape[0] - total.shape[0])]).contiguous()
         if self.conv_taps:
             taps = [tensors["q_conv"]] + ([] if self.shared_kv else [tensors["k_conv"], tensors["v_conv"]])
             self.conv = torch.cat([t.to(taps[0].dtype) for t in taps]).contiguous()
@@ -216,6 +234,8 @@ class Attention:
                 kw["norm_bare"] = True
             if self.qk_norm_last:
                 kw["norm_last"] = True
+            if self.qkv_bias is not None:
+                kw["bias"] = self.qkv_bias
             # values that are the keys as projected: the value columns of the row are its key columns
             ops.qkv_prepare(src, partials, (0, H * d, H * d if self.values_are_keys else (H + G) * d), q, view.kv, batch, H, G, d, dv,
                             table=None if pos is None else pos.table, rot_dims=0 if pos is None else pos.head_dim,

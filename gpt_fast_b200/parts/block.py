@@ -3,7 +3,8 @@
 residual stream x kept in 32-bit, optionally with a learned factor per column on each
 sublayer and a token input behind them.  'sandwich' norms a sublayer's output as well
 and scales it before the sum; its feed-forward is optional.  'parallel' runs mixer and
-feed-forward side by side on two norms of the same x.
+feed-forward side by side on two norms of the same x.  'streams' is the pre-norm arrangement
+over several residual streams.
 
 An arrangement declares `roles`: the names of the parts it is made of, each with
 the kind of part that fills it ('mixer', 'feed_forward', 'norm': the registries of
@@ -14,6 +15,7 @@ import torch
 from ..weights.loader import ParamSpec
 from . import register_block
 from .residual import Branch, as_residual
+from .streams import StreamMix, Streams
 
 
 @register_block("prenorm")
@@ -63,6 +65,49 @@ class PreNormBlock:
                 x.add_scaled(y, self.ffn_scale.weight)
         if self.token_input is not None:
             self.token_input.forward(x, batch)
+
+
+@register_block("streams")
+class StreamsBlock:
+    """The pre-norm arrangement over n residual streams (`parts.streams`): per sublayer, with its constants enter, leave and mix,
+
+        u = sum_s enter_s x_s;   y = sublayer(norm(u));   x_t <- sum_s mix_st x_s + leave_t y
+
+    The feed-forward (with its norm and constants) is optional.  A sublayer writes into a `Branch`; the update is left to the
+    streams, whose next reader does it on the way."""
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "mixer_norm": "norm", "ffn_norm": "norm"}
+    optional_roles = ("feed_forward", "ffn_norm")
+    takes_streams = True
+
+    def __init__(self, parts: dict, dim: int, dtype: torch.dtype, streams: int):
+        if ("feed_forward" in parts) != ("ffn_norm" in parts):
+            raise ValueError("a block of streams has a feed-forward with its norm or neither")
+        self._parts = dict(parts)
+        self.mixer, self.mixer_norm = parts["mixer"], parts["mixer_norm"]
+        self.feed_forward, self.ffn_norm = parts.get("feed_forward"), parts.get("ffn_norm")
+        self.dim, self.dtype = dim, dtype
+        self.mixer_streams = self._parts["mixer_streams"] = StreamMix(streams)
+        self.ffn_streams = None
+        if self.feed_forward is not None:
+            self.ffn_streams = self._parts["ffn_streams"] = StreamMix(streams)
+
+    def parts(self):
+        return dict(self._parts)
+
+    def cache_needs(self):
+        return self.mixer.cache_needs()
+
+    def forward(self, x: Streams, batch, view, append: bool = True):
+        h = torch.empty(x.n_tokens, self.dim, dtype=self.dtype, device=x.device)
+        self.mixer_norm.forward(x.read(self.mixer_streams), h)
+        y = Branch(x.n_tokens, self.dim, x.device)
+        self.mixer.forward(h, batch, view, residual=y, append=append)
+        x.leave(y, self.mixer_streams)
+        if self.feed_forward is not None:
+            self.ffn_norm.forward(x.read(self.ffn_streams), h)
+            y = Branch(x.n_tokens, self.dim, x.device)
+            self.feed_forward.forward(h, residual=y)
+            x.leave(y, self.ffn_streams)
 
 
 @register_block("sandwich")

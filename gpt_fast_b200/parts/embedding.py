@@ -8,7 +8,10 @@ with the table's last row (number `buckets`) for a sequence's first token.  The 
 state (one int32 in the cache), so a sequence may arrive in portions of any size.
 
 'learned_position': a learned vector per position, x_t = table[tok_t] + positions[p_t], p_t counted from 0 in each
-sequence; it keeps no state (a token's position is its sequence's cached length plus its place in the step)."""
+sequence; it keeps no state (a token's position is its sequence's cached length plus its place in the step).
+
+'normed': nothing is added, but the embedding passes a root-mean-square norm, x_t = e / sqrt(mean(e^2) + eps) * w, e =
+table[tok_t]."""
 import torch
 
 from .. import ops
@@ -40,6 +43,29 @@ class BigramHash:
     def forward(self, tokens, table, out, batch, view, scale: float = 1.0):
         """out float32 [T, dim] = table[tokens] * scale + the hashed rows; view.state int32 [n_slots, 1]."""
         ops.embed_hashed(tokens, table, self.table, out, batch, view.state.view(-1), self.buckets, self.mul_prev, self.mul_cur, scale)
+
+
+@register_embedding("normed")
+class NormedEmbedding:
+    def __init__(self, dim: int, eps: float, dtype: torch.dtype):
+        self.dim, self.eps, self.dtype = dim, float(eps), dtype
+        self.weight = None
+
+    def param_specs(self):
+        return {"weight": ParamSpec((self.dim,), "vector")}
+
+    def load(self, tensors):
+        self.weight = tensors["weight"]
+
+    def export(self):
+        return {"weight": self.weight}
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds()
+
+    def forward(self, tokens, table, out, batch, view, scale: float = 1.0):
+        """out float32 [T, dim] = norm(table[tokens] * scale)."""
+        ops.embed_normed(tokens, table, self.weight, self.eps, out, batch.status, scale)
 
 
 @register_embedding("learned_position")

@@ -12,8 +12,9 @@ plain SwiGLU that every token runs; with `shared_gate` its output is multiplied 
 whose row rides behind the router's rows in one product.
 
 Score 'softmax' takes s = softmax(z) over all experts, chooses by s + correction and weighs by s * scale as it is.
-`groups` = (count, keep): the experts are `count` equal groups of neighbours; a group's score is the largest choice score in it
-and only experts of the `keep` best groups can be chosen.  `activation` 'relu2': experts (and the shared one) of two products,
+Score 'sigmoid_plain' is 'sigmoid' with the chosen experts' s * scale as weights, not divided by their sum.
+`groups` = (count, keep[, terms]): the experts are `count` equal groups of neighbours; a group's score is the largest choice score
+in it (with terms = 2 the sum of its two largest) and only experts of the `keep` best groups can be chosen.  `activation` 'relu2': experts (and the shared one) of two products,
 W_down max(W_up h, 0)^2.  A shared expert without a gate and of the experts' own size is one more expert that every token
 chooses with weight 1, so the experts' products run it along; of another size it is a feed-forward of its own.
 
@@ -40,19 +41,23 @@ class MixtureOfExperts:
                  shared_hidden: int = 0, shared_gate: bool = False, activation: str = "glu", groups=None):
         if not 1 <= top <= n_experts:
             raise ValueError(f"{top} of {n_experts} experts per token")
-        if score not in ("sigmoid", "softmax_top", "softmax"):
-            raise ValueError(f"a router score is 'sigmoid', 'softmax_top' or 'softmax', not {score!r}")
+        if score not in ("sigmoid", "sigmoid_plain", "softmax_top", "softmax"):
+            raise ValueError(f"a router score is 'sigmoid', 'sigmoid_plain', 'softmax_top' or 'softmax', not {score!r}")
         if activation not in ("glu", "relu2"):
             raise ValueError(f"the experts' activation is 'glu' or 'relu2', not {activation!r}")
         if groups is not None and (groups[0] < 1 or n_experts % groups[0] or not 1 <= groups[1] <= groups[0]
                                    or top > groups[1] * (n_experts // groups[0])):
             raise ValueError(f"{top} experts from {groups[1]} of {groups[0]} groups of {n_experts} experts in all")
-        self.activation, self.groups = activation, None if groups is None or groups[0] == 1 else (int(groups[0]), int(groups[1]))
+        if groups is not None and len(groups) > 2 and groups[2] not in (1, 2):
+            raise ValueError(f"a group's score is made of one or two choice scores, not {groups[2]}")
+        self.activation, self.groups = activation, None if groups is None or groups[0] == 1 else tuple(int(g) for g in groups)
         if shared_gate and not shared_hidden:
             raise ValueError("a gate for a shared expert that is not there")
         self.score, self.shared_hidden, self.shared_gate = score, int(shared_hidden or 0), bool(shared_gate)
         # one more expert that every token chooses, in the experts' own stacks
-        self.shared_inside = bool(self.shared_hidden) and not self.shared_gate and activation == "relu2" and self.shared_hidden == hidden
+        plain_glu = float(limit) <= 0 and float(alpha) == 1.0 and float(shift) == 0.0          # the shared expert is a plain SwiGLU
+        self.shared_inside = (bool(self.shared_hidden) and not self.shared_gate and self.shared_hidden == hidden
+                              and (activation == "relu2" or plain_glu))
         self.shared_w13 = self.shared_w2 = None
         self.dim, self.hidden, self.n_experts, self.top, self.dtype = dim, hidden, int(n_experts), int(top), dtype
         self.router_scale, self.limit, self.alpha, self.shift = float(router_scale), float(limit), float(alpha), float(shift)
@@ -94,6 +99,9 @@ class MixtureOfExperts:
         # rows alternate gate, up within every expert
         self.w13 = torch.stack([tensors["gate"], tensors["up"]], dim=2).reshape(E, 2 * F, D).contiguous()
         self.w2 = tensors["down"]
+        if self.shared_inside:
+            self.w13, self.w2 = torch.cat([self.w13, self.shared_w13[None]]), torch.cat([self.w2, self.shared_w2[None]])
+            self.shared_w13 = self.shared_w2 = None
 
     def export(self):
         if self.activation == "relu2":
@@ -107,13 +115,14 @@ class MixtureOfExperts:
                 if self.shared_gate:
                     out["shared_sg"] = self.router[E:E + 1]
             return out
-        w = self.w13.view(self.n_experts, self.hidden, 2, self.dim)
-        out = {"router": self._router_stored, "gate": w[:, :, 0], "up": w[:, :, 1], "down": self.w2}
+        E = self.n_experts
+        w = self.w13.view(-1, self.hidden, 2, self.dim)
+        out = {"router": self._router_stored, "gate": w[:E, :, 0], "up": w[:E, :, 1], "down": self.w2[:E]}
         if self.has_correction:
             out["correction"] = self.correction
         if self.shared_hidden:
-            sw = self.shared_w13.view(self.shared_hidden, 2, self.dim)
-            out.update(shared_gate=sw[:, 0], shared_up=sw[:, 1], shared_down=self.shared_w2)
+            sw = w[E] if self.shared_inside else self.shared_w13.view(self.shared_hidden, 2, self.dim)
+            out.update(shared_gate=sw[:, 0], shared_up=sw[:, 1], shared_down=self.w2[E] if self.shared_inside else self.shared_w2)
             if self.shared_gate:
                 out["shared_sg"] = self.router[self.n_experts:self.n_experts + 1]
         return out

@@ -7,6 +7,7 @@ from .. import ops
 from ..weights.loader import ParamSpec
 from . import register_norm
 from .residual import Residual
+from .streams import StreamRead
 
 
 def _owed_scaled(x: Residual, rows):
@@ -49,8 +50,11 @@ class RMSNorm:
         """x: the residual stream (a `Residual`, or a complete float32 tensor
         [T, dim]) -> out [R, dim] in the compute dtype; `rows` (int32 [R]) picks
         input rows, else R = T.  Partial sums pending on the stream are added
-        by the same kernel, and so are a branch with a root-mean-square norm of its own or scaled branches."""
-        if isinstance(x, Residual):
+        by the same kernel, and so are a branch with a root-mean-square norm of its own or scaled branches.  A weighted sum of
+        several streams (a `StreamRead`) is made, and the update they are owed done, by the same kernel as well."""
+        if isinstance(x, StreamRead):
+            x.into(out, self.weight, self.eps, rows)
+        elif isinstance(x, Residual):
             branch = _owed_rms_branch(x, rows)
             scaled = _owed_scaled(x, rows) if branch is None else None
             if branch is not None:
@@ -86,7 +90,9 @@ class NoNorm:
         return {}
 
     def forward(self, x, out, rows=None):
-        if isinstance(x, Residual):
+        if isinstance(x, StreamRead):
+            x.into(out, rows=rows)
+        elif isinstance(x, Residual):
             branch = _owed_rms_branch(x, rows)
             scaled = _owed_scaled(x, rows) if branch is None else None
             if branch is not None:
@@ -134,6 +140,8 @@ class LayerNorm:
     def forward(self, x, out, rows=None):
         """x: the residual stream (a `Residual`, or a complete float32 tensor [T, dim]) -> out [R, dim] in the
         compute dtype; `rows` (int32 [R]) picks input rows."""
+        if isinstance(x, StreamRead):
+            x = x.value()
         if not isinstance(x, Residual):
             ops.layernorm(x, self.weight, self.bias, self.eps, out, rows)
             return out

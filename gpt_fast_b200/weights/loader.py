@@ -126,6 +126,10 @@ class RandomCheckpoint:
             x = (1.0 + x * self.jitter).to(self.vector_dtype)
         elif s.init == "bias":
             x = (x * self.jitter).to(self.vector_dtype)
+        elif s.init == "share":
+            x = (1.0 / s.shape[0] + x * self.jitter).to(self.vector_dtype)
+        elif s.init == "identity":
+            x = (torch.eye(s.shape[0], device=x.device) + x * self.jitter).to(self.vector_dtype)
         elif s.init == "unit":
             x = x.to(self.vector_dtype)
         elif s.init == "conv":

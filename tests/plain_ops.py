@@ -69,6 +69,28 @@ class PlainOps:
         out.copy_(table[ids.clamp(0, table.shape[0] - 1)].float() * scale)
         out[bad] = 0
 
+    def embed_normed(self, tokens, table, weight, eps, out, status, scale=1.0):
+        self.embed(tokens, table, out, status, scale)
+        e = out.double()
+        out.copy_((e * torch.rsqrt((e * e).mean(-1, keepdim=True) + eps) * weight.double()).float())
+
+    def streams(self, x, n, shared=False, x_out=None, mix=None, leave=None, branches=(), enter=None, weight=None, eps=0.0, out=None,
+                rows=None):
+        v = (x.expand(n, *x.shape) if shared else x).double()
+        if mix is not None:
+            y = sum((b.double().sum(0) if b.dim() == 3 else b.double()) for b in branches) if branches else torch.zeros_like(v[0])
+            v = torch.stack([sum(float(mix[s, t]) * v[s] for s in range(n)) + float(leave[t]) * y for t in range(n)])
+            if x_out is not None:
+                x_out.copy_(v.float())
+        if out is None:
+            return
+        u = sum((1.0 if enter is None else float(enter[t])) * v[t] for t in range(n))
+        if rows is not None:
+            u = u[rows.long()]
+        if weight is not None:
+            u = u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps) * weight.double()
+        out.copy_(u.to(out.dtype))
+
     def embed_positions(self, tokens, table, positions, out, batch, scale=1.0):
         pos, _ = token_positions(batch)
         if int(pos.max()) >= positions.shape[0]:
@@ -84,19 +106,20 @@ class PlainOps:
     def moe_route(self, logits, correction, top, scale, idx, weights, score="sigmoid", groups=(1, 1), shared=False):
         E = correction.shape[0]
         z = logits[:, :E].float()
-        s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z.double(), -1).float() if score == "softmax" else z
+        s = torch.sigmoid(z) if score in ("sigmoid", "sigmoid_plain") else torch.softmax(z.double(), -1).float() if score == "softmax" else z
         choice = s + correction.float()
         per = E // groups[0]
         if shared:
             idx[:, top], weights[:, top] = E, 1.0
             idx, weights = idx[:, :top], weights[:, :top]
         for t in range(s.shape[0]):
-            best = [float(choice[t, g * per:(g + 1) * per].max()) for g in range(groups[0])]
+            terms = groups[2] if len(groups) > 2 else 1
+            best = [float(choice[t, g * per:(g + 1) * per].sort(descending=True).values[:terms].double().sum()) for g in range(groups[0])]
             kept = set(sorted(range(groups[0]), key=lambda g: (-best[g], g))[:groups[1]])
             order = sorted((e for e in range(E) if e // per in kept), key=lambda e: (-float(choice[t, e]), e))[:top]
             picked = s[t, order]
             idx[t] = torch.tensor(order, dtype=idx.dtype)
-            if score == "softmax":
+            if score in ("softmax", "sigmoid_plain"):
                 weights[t] = picked * scale
             elif score == "sigmoid":
                 weights[t] = picked / (picked.sum() + 1e-20) * scale
@@ -339,10 +362,13 @@ class PlainOps:
 
     def qkv_prepare(self, src, partials, offsets, q_out, kv, batch, n_head, n_kv, head_dim, v_head_dim, table=None, rot_dims=0,
                     pairing="half", q_norm=None, k_norm=None, norm_eps=0.0, k_scale=1.0, append=True, norm_whole=False,
-                    norm_bare=False, norm_last=False, maps=1):
+                    norm_bare=False, norm_last=False, maps=1, q_spread=False, bias=None):
+        assert not q_spread                                    # a layout of the tensor-core kernels only
         H, G, d, dv = n_head * maps, n_kv * maps, head_dim, v_head_dim
         T = batch.n_tokens
         x = (partials.double().sum(0) if partials is not None else src.double())
+        if bias is not None:
+            x = x + bias.double()
         qo, ko, vo = offsets
         q = x[:, qo:qo + H * d].reshape(T, H, d)
         if append:
