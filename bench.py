@@ -418,6 +418,13 @@ def design_bench(a, design):
     # channel, and its other design of three routed experts and a shared one of 1792, both at the same width, depth and vocabulary
     tables["dufizen"] = [("dufizen-1b", a.layers, "gikepel", lambda cfg: config_from_name("gikepel-1b"),
                           "tapupel", lambda cfg: config_from_name("tapupel-1b"))]
+    # beside Pikalix: the library's other designs of windowed attention (one with readers of another layer's keys and a q/k norm over
+    # the whole projection, one with three routed experts and a shared one of 1792), at the same width, depth, heads, head size,
+    # window and vocabulary
+    tables["pikalix"] = [("pikalix-1b", a.layers, "tapupel", lambda cfg: dict(config_from_name("tapupel-1b"),
+                                                                             layers=config_from_name("tapupel-1b")["layers"][:len(cfg["layers"])]),
+                          "lomusun", lambda cfg: dict(config_from_name("lomusun-1b"),
+                                                      layers=config_from_name("lomusun-1b")["layers"][:len(cfg["layers"])]))]
     if design not in tables:
         print(f"bench.py: no size table for design '{design}'")
         return 2
@@ -469,7 +476,7 @@ def main():
     ap.add_argument("--skip-configs", action="store_true", help="leave out the Llama-3.2-3B and Llama-2-13B sizes")
     ap.add_argument("--skip-shares", action="store_true", help="leave out the per-kernel shares")
     ap.add_argument("--design", default=None, help="instead of the default workload: prefill and decode of another design "
-                    "(lasezen, gikepel, lomusun, tapupel, dufizen) at layer sizes of a real model, beside the library's closest other model at equal size")
+                    "(lasezen, gikepel, lomusun, tapupel, dufizen, pikalix) at layer sizes of a real model, beside the library's closest other model at equal size")
     ap.add_argument("--design-model", default=None, help=argparse.SUPPRESS)       # one model of --design, run as a child process
     ap.add_argument("--design-label", default="model", help=argparse.SUPPRESS)
     ap.add_argument("--prefill-lengths", default=None, help="with --design: prompt lengths of the prefill rows (default 512,2048,8192)")

@@ -15,7 +15,8 @@
 // key row holds the `maps` vectors of its head one after the other.
 // A projection's biases (one number per column of the source row) are added ahead of everything else.
 // One warp per (token, head), the head in shared memory between the steps; with a norm over the whole projection one
-// block per token, the token's q, k and v in shared memory between the steps, so every number is read once.
+// block per token, the token's q, k and v in registers (or, where a rotation pairs numbers of different threads, in shared
+// memory) between the steps, so every number is read once.
 #include "common.cuh"
 
 GFB_DEFINE_LAST_ERROR()
@@ -256,6 +257,116 @@ __global__ void qkv_prepare_token_kernel(const void* __restrict__ src, int S, si
     }
 }
 
+// The same with the token's numbers in registers, NP packs of four per thread: for rotations whose pairs are neighbours (or none),
+// where nothing a thread needs lies with another one but the two mean squares.
+template <typename T, int NP>
+__global__ void qkv_prepare_regs_kernel(const void* __restrict__ src, int S, size_t slice, int width, int q_off, int k_off, int v_off,
+                                        const void* __restrict__ bias, int b_dt, T* __restrict__ q_out, GfbPagedKV kv, GfbBatch b,
+                                        const float* __restrict__ table, int table_len, int rot_dims, const void* q_norm, const void* k_norm,
+                                        int w_dt, float eps, float k_scale, int H, int G, int dk, int dv, int append, int* status) {
+    __shared__ float2 scratch[32];
+    const int nq = H * dk, nk = append ? G * dk : 0, nv = append ? G * dv : 0;
+    const int packs = (nq + nk + nv) >> 2;
+    gfb_pdl_launch();
+    gfb_pdl_wait();
+    const int t = blockIdx.x;
+    const int s = b.tok_seq[t];
+    const int slot = b.slots[s];
+    const int pos = b.lengths[slot] + (t - b.cu_seqlens[s]);
+    const size_t row = (size_t)t * width;
+    float x[NP][4];
+    float2 ss = make_float2(0.f, 0.f);                              // q's and k's sums of squares
+#pragma unroll
+    for (int p = 0; p < NP; p++) {
+        const int i = 4 * (threadIdx.x + p * blockDim.x);           // the pack's place in q, k, v one behind the other
+        if (i >= 4 * packs) continue;
+        const int c = i < nq ? q_off + i : i < nq + nk ? k_off + i - nq : v_off + i - nq - nk;
+        if (S > 0) {
+            const float* f = (const float*)src + row + c;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            constexpr int W = NP == 1 ? 8 : 4;                      // partial sums in flight together, added in ascending order
+            for (int k = 0; k < S; k += W) {
+                float4 a[W];
+#pragma unroll
+                for (int u = 0; u < W; u++) a[u] = *reinterpret_cast<const float4*>(f + (size_t)min(k + u, S - 1) * slice);
+#pragma unroll
+                for (int u = 0; u < W; u++)
+                    if (k + u < S) { v.x += a[u].x; v.y += a[u].y; v.z += a[u].z; v.w += a[u].w; }
+            }
+            x[p][0] = v.x; x[p][1] = v.y; x[p][2] = v.z; x[p][3] = v.w;
+        } else {
+            const AlignedPack<T, 4> a = *reinterpret_cast<const AlignedPack<T, 4>*>((const T*)src + row + c);
+#pragma unroll
+            for (int e = 0; e < 4; e++) x[p][e] = gfb_to_f32(a.v[e]);
+        }
+        float sum = 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            if (bias != nullptr) x[p][e] += ld_w(bias, b_dt, c + e);
+            sum += x[p][e] * x[p][e];
+        }
+        if (i < nq) ss.x += sum;
+        else if (i < nq + nk) ss.y += sum;
+    }
+    bool ok = pos >= 0 && (table == nullptr || pos < table_len);
+    int page = -1, off = 0;
+    if (append && ok) {
+        const int pi = pos / kv.page_size;
+        off = pos - pi * kv.page_size;
+        page = pi < kv.max_pages ? kv.page_table[(size_t)slot * kv.max_pages + pi] : -1;
+        ok = page >= 0 && page < kv.n_pages;
+    }
+    if (!ok) {                                                      // the same for every thread of the block
+        if (threadIdx.x == 0) gfb_report(status, GFB_ERR_CACHE_RANGE, t, pos);
+        for (int i = threadIdx.x; i < nq; i += blockDim.x) q_out[(size_t)t * nq + i] = gfb_from_f32<T>(0.f);     // q stays defined
+        return;
+    }
+    {
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+        ss.x = gfb_warp_sum(ss.x);
+        ss.y = gfb_warp_sum(ss.y);
+        if (lane == 0) scratch[warp] = ss;
+        __syncthreads();
+        ss = lane < nwarp ? scratch[lane] : make_float2(0.f, 0.f);
+        ss.x = gfb_warp_sum(ss.x);
+        ss.y = gfb_warp_sum(ss.y);
+    }
+    const float rq = q_norm != nullptr ? 1.0f / sqrtf(ss.x / (float)nq + eps) : 1.f;
+    const float rk = k_norm != nullptr ? 1.0f / sqrtf(ss.y / (float)max(nk, 1) + eps) : 1.f;
+    const float* cs = table != nullptr ? table + (size_t)pos * rot_dims : nullptr;
+#pragma unroll
+    for (int p = 0; p < NP; p++) {
+        const int i = 4 * (threadIdx.x + p * blockDim.x);
+        if (i >= 4 * packs) continue;
+        const bool is_q = i < nq, is_k = !is_q && i < nq + nk;
+        const int at = is_q ? i : is_k ? i - nq : i - nq - nk;      // place in q, k or v
+        const int d = is_q || is_k ? dk : dv, head = at / d, j = at - head * d;
+        T* dst;
+        if (is_q) dst = q_out + (size_t)t * nq + at;
+        else dst = (T*)(is_k ? kv.k_pool : kv.v_pool) + (((size_t)page * G + head) * kv.page_size + off) * d + j;
+        if (is_q || is_k) {
+            const void* w = is_q ? q_norm : k_norm;
+            const float r = is_q ? rq : rk, f = is_q ? 1.f : k_scale;
+#pragma unroll
+            for (int e = 0; e < 4; e++) x[p][e] *= r * (w != nullptr ? ld_w(w, w_dt, at + e) : 1.f);
+#pragma unroll
+            for (int e = 0; e < 4; e += 2)
+                if (j + e < rot_dims) {
+                    const float2 turn = *reinterpret_cast<const float2*>(cs + j + e);
+                    const float u = x[p][e], v = x[p][e + 1];
+                    x[p][e] = u * turn.x - v * turn.y;
+                    x[p][e + 1] = v * turn.x + u * turn.y;
+                }
+#pragma unroll
+            for (int e = 0; e < 4; e++) x[p][e] *= f;
+        }
+        AlignedPack<T, 4> o;
+#pragma unroll
+        for (int e = 0; e < 4; e++) o.v[e] = gfb_from_f32<T>(x[p][e]);
+        *reinterpret_cast<AlignedPack<T, 4>*>(dst) = o;
+    }
+}
+
 template <typename T, int N, typename... A>
 static cudaError_t launch_token(size_t smem, int n_tokens, int threads, cudaStream_t stream, A... args) {
     if (smem > 40 * 1024) {
@@ -297,6 +408,26 @@ GFB_API int gfb_qkv_prepare(const void* src, int n_partials, int width, int q_of
         const bool four = ((q_off | k_off | v_off | width | dk | dv) & 3) == 0
                           && (((uintptr_t)src | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) == 0;
         const long cols = (long)H * dk + (append ? (long)G * (dk + dv) : 0);
+        if (four && (table == nullptr || pairing == 0) && cols <= 16384) {
+            // few tokens: as many threads as packs (a token's latency is what counts); many: up to four packs per thread
+            const int packs = (int)(cols / 4);
+            const int most = n_tokens <= 128 ? 1024 : 256;
+            int np = (packs + most - 1) / most;
+            np = np <= 1 ? 1 : np <= 2 ? 2 : np <= 4 ? 4 : 8;
+            const int threads = ((packs + np - 1) / np + 31) / 32 * 32;
+            if (threads <= (np == 8 ? 512 : 1024)) {
+#define REGS(T, NP) e = gfb_launch(qkv_prepare_regs_kernel<T, NP>, dim3((unsigned)n_tokens), dim3((unsigned)threads), 0, stream, src, n_partials, slice, width, \
+                                   q_off, k_off, v_off, bias, b_dt, (T*)q_out, kv, b, table, table_len, table != nullptr ? rot_dims : 0, q_norm, k_norm, w_dt, eps, \
+                                   k_scale, H, G, dk, dv, append, status)
+#define REGS_NP(T) do { if (np == 1) REGS(T, 1); else if (np == 2) REGS(T, 2); else if (np == 4) REGS(T, 4); else REGS(T, 8); } while (0)
+                if (dt == GFB_BF16) REGS_NP(__nv_bfloat16);
+                else if (dt == GFB_F32) REGS_NP(float);
+                else return gfb_fail("gfb_qkv_prepare: unknown type %d", dt);
+#undef REGS_NP
+#undef REGS
+                return gfb_check(e, "gfb_qkv_prepare (registers)");
+            }
+        }
         const int threads = cols <= 1024 ? 128 : n_tokens <= 128 && cols > 2048 ? 512 : 256;
 #define TOKEN(T, N) e = launch_token<T, N>(token_smem, n_tokens, threads, stream, src, n_partials, slice, width, q_off, k_off, v_off, bias, b_dt, \
                                            (T*)q_out, kv, b, table, table_len, table != nullptr ? rot_dims : 0, pairing, q_norm, k_norm, w_dt, eps, k_scale, H, G, \
