@@ -258,113 +258,185 @@ __global__ void qkv_prepare_token_kernel(const void* __restrict__ src, int S, si
 }
 
 // The same with the token's numbers in registers, NP packs of four per thread: for rotations whose pairs are neighbours (or none),
-// where nothing a thread needs lies with another one but the two mean squares.
+// where nothing a thread needs lies with another one but the two mean squares.  A block takes every gridDim.x-th token; a thread's
+// columns, and with them its biases and norm weights, are the same for all of them and are fetched once.
+__device__ __forceinline__ void ld_w4(float (&v)[4], const void* p, int dt, int i) {          // i: a multiple of four
+    if (dt == GFB_BF16) {
+        const AlignedPack<__nv_bfloat16, 4> a = *reinterpret_cast<const AlignedPack<__nv_bfloat16, 4>*>((const __nv_bfloat16*)p + i);
+#pragma unroll
+        for (int e = 0; e < 4; e++) v[e] = __bfloat162float(a.v[e]);
+    } else {
+        const float4 a = *reinterpret_cast<const float4*>((const float*)p + i);
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    }
+}
+
+constexpr int regs_threads(int np) { return np == 1 ? 1024 : np == 2 ? 768 : 640; }      // the largest block whose registers suffice
+
 template <typename T, int NP>
-__global__ void qkv_prepare_regs_kernel(const void* __restrict__ src, int S, size_t slice, int width, int q_off, int k_off, int v_off,
+__global__ void __launch_bounds__(regs_threads(NP)) qkv_prepare_regs_kernel(const void* __restrict__ src, int S, size_t slice, int width, int q_off, int k_off, int v_off,
                                         const void* __restrict__ bias, int b_dt, T* __restrict__ q_out, GfbPagedKV kv, GfbBatch b,
                                         const float* __restrict__ table, int table_len, int rot_dims, const void* q_norm, const void* k_norm,
                                         int w_dt, float eps, float k_scale, int H, int G, int dk, int dv, int append, int* status) {
-    __shared__ float2 scratch[32];
+    __shared__ float2 scratch[2][32];
     const int nq = H * dk, nk = append ? G * dk : 0, nv = append ? G * dv : 0;
-    const int packs = (nq + nk + nv) >> 2;
+    const int cols = nq + nk + nv;
     gfb_pdl_launch();
-    gfb_pdl_wait();
-    const int t = blockIdx.x;
-    const int s = b.tok_seq[t];
-    const int slot = b.slots[s];
-    const int pos = b.lengths[slot] + (t - b.cu_seqlens[s]);
-    const size_t row = (size_t)t * width;
-    float x[NP][4];
-    float2 ss = make_float2(0.f, 0.f);                              // q's and k's sums of squares
-#pragma unroll
-    for (int p = 0; p < NP; p++) {
-        const int i = 4 * (threadIdx.x + p * blockDim.x);           // the pack's place in q, k, v one behind the other
-        if (i >= 4 * packs) continue;
-        const int c = i < nq ? q_off + i : i < nq + nk ? k_off + i - nq : v_off + i - nq - nk;
-        if (S > 0) {
-            const float* f = (const float*)src + row + c;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            constexpr int W = NP == 1 ? 8 : 4;                      // partial sums in flight together, added in ascending order
-            for (int k = 0; k < S; k += W) {
-                float4 a[W];
-#pragma unroll
-                for (int u = 0; u < W; u++) a[u] = *reinterpret_cast<const float4*>(f + (size_t)min(k + u, S - 1) * slice);
-#pragma unroll
-                for (int u = 0; u < W; u++)
-                    if (k + u < S) { v.x += a[u].x; v.y += a[u].y; v.z += a[u].z; v.w += a[u].w; }
-            }
-            x[p][0] = v.x; x[p][1] = v.y; x[p][2] = v.z; x[p][3] = v.w;
-        } else {
-            const AlignedPack<T, 4> a = *reinterpret_cast<const AlignedPack<T, 4>*>((const T*)src + row + c);
-#pragma unroll
-            for (int e = 0; e < 4; e++) x[p][e] = gfb_to_f32(a.v[e]);
-        }
-        float sum = 0.f;
-#pragma unroll
-        for (int e = 0; e < 4; e++) {
-            if (bias != nullptr) x[p][e] += ld_w(bias, b_dt, c + e);
-            sum += x[p][e] * x[p][e];
-        }
-        if (i < nq) ss.x += sum;
-        else if (i < nq + nk) ss.y += sum;
-    }
-    bool ok = pos >= 0 && (table == nullptr || pos < table_len);
-    int page = -1, off = 0;
-    if (append && ok) {
-        const int pi = pos / kv.page_size;
-        off = pos - pi * kv.page_size;
-        page = pi < kv.max_pages ? kv.page_table[(size_t)slot * kv.max_pages + pi] : -1;
-        ok = page >= 0 && page < kv.n_pages;
-    }
-    if (!ok) {                                                      // the same for every thread of the block
-        if (threadIdx.x == 0) gfb_report(status, GFB_ERR_CACHE_RANGE, t, pos);
-        for (int i = threadIdx.x; i < nq; i += blockDim.x) q_out[(size_t)t * nq + i] = gfb_from_f32<T>(0.f);     // q stays defined
-        return;
-    }
-    {
-        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
-        ss.x = gfb_warp_sum(ss.x);
-        ss.y = gfb_warp_sum(ss.y);
-        if (lane == 0) scratch[warp] = ss;
-        __syncthreads();
-        ss = lane < nwarp ? scratch[lane] : make_float2(0.f, 0.f);
-        ss.x = gfb_warp_sum(ss.x);
-        ss.y = gfb_warp_sum(ss.y);
-    }
-    const float rq = q_norm != nullptr ? 1.0f / sqrtf(ss.x / (float)nq + eps) : 1.f;
-    const float rk = k_norm != nullptr ? 1.0f / sqrtf(ss.y / (float)max(nk, 1) + eps) : 1.f;
-    const float* cs = table != nullptr ? table + (size_t)pos * rot_dims : nullptr;
+    // what a pack is, the same for every token: its column in the source row (from), its place in a token's q or, head by head, in
+    // its page of keys or values (to), its place in its head (in_head), and its constants
+    enum { IS_Q = 0, IS_K = 1, IS_V = 2, NONE = 3 };
+    float wt[NP][4], bi[NP][4];
+    int kind[NP], from[NP], to[NP], in_head[NP];
 #pragma unroll
     for (int p = 0; p < NP; p++) {
         const int i = 4 * (threadIdx.x + p * blockDim.x);
-        if (i >= 4 * packs) continue;
-        const bool is_q = i < nq, is_k = !is_q && i < nq + nk;
-        const int at = is_q ? i : is_k ? i - nq : i - nq - nk;      // place in q, k or v
-        const int d = is_q || is_k ? dk : dv, head = at / d, j = at - head * d;
-        T* dst;
-        if (is_q) dst = q_out + (size_t)t * nq + at;
-        else dst = (T*)(is_k ? kv.k_pool : kv.v_pool) + (((size_t)page * G + head) * kv.page_size + off) * d + j;
-        if (is_q || is_k) {
-            const void* w = is_q ? q_norm : k_norm;
-            const float r = is_q ? rq : rk, f = is_q ? 1.f : k_scale;
+        kind[p] = i < nq ? IS_Q : i < nq + nk ? IS_K : i < cols ? IS_V : NONE;
+        from[p] = to[p] = in_head[p] = 0;
 #pragma unroll
-            for (int e = 0; e < 4; e++) x[p][e] *= r * (w != nullptr ? ld_w(w, w_dt, at + e) : 1.f);
+        for (int e = 0; e < 4; e++) { wt[p][e] = 1.f; bi[p][e] = 0.f; }
+        if (kind[p] == NONE) continue;
+        const int at = kind[p] == IS_Q ? i : kind[p] == IS_K ? i - nq : i - nq - nk, d = kind[p] == IS_V ? dv : dk;
+        const int head = at / d;
+        in_head[p] = at - head * d;
+        to[p] = kind[p] == IS_Q ? at : head * kv.page_size * d + in_head[p];
+        from[p] = (kind[p] == IS_Q ? q_off : kind[p] == IS_K ? k_off : v_off) + at;
+        if (kind[p] == IS_Q && q_norm != nullptr) ld_w4(wt[p], q_norm, w_dt, at);
+        if (kind[p] == IS_K && k_norm != nullptr) ld_w4(wt[p], k_norm, w_dt, at);
+        if (kind[p] == IS_V) in_head[p] = rot_dims;                 // values are not rotated
+        if (bias != nullptr) ld_w4(bi[p], bias, b_dt, from[p]);
+    }
+    gfb_pdl_wait();
+    // Where a token goes: a chain of four dependent loads, so one warp looks up the block's next 32 tokens at a time.  What a token
+    // brings is fetched while the block still works on the one before it.
+    struct Place { int pos, page, off, ok; };
+    __shared__ Place places[32];
+    auto look_up = [&](int first) {
+        const int t = first + (int)threadIdx.x * (int)gridDim.x;
+        if (threadIdx.x >= 32 || t >= b.n_tokens) return;
+        Place a;
+        const int s = b.tok_seq[t];
+        const int slot = b.slots[s];
+        a.pos = b.lengths[slot] + (t - b.cu_seqlens[s]);
+        a.ok = a.pos >= 0 && (table == nullptr || a.pos < table_len);
+        a.page = -1;
+        a.off = 0;
+        if (append && a.ok) {
+            const int pi = a.pos / kv.page_size;
+            a.off = a.pos - pi * kv.page_size;
+            a.page = pi < kv.max_pages ? kv.page_table[(size_t)slot * kv.max_pages + pi] : -1;
+            a.ok = a.page >= 0 && a.page < kv.n_pages;
+        }
+        if (!a.ok) gfb_report(status, GFB_ERR_CACHE_RANGE, t, a.pos);
+        places[threadIdx.x] = a;
+    };
+    AlignedPack<T, 4> raw[NP] = {};                                  // (zeros where there is no pack)
+    auto fetch = [&](int t) {
+        if (S > 0) return;
+        const T* row = (const T*)src + (size_t)t * width;
+#pragma unroll
+        for (int p = 0; p < NP; p++)
+            if (kind[p] != NONE) raw[p] = *reinterpret_cast<const AlignedPack<T, 4>*>(row + from[p]);
+    };
+    fetch(blockIdx.x);                                               // (a block has at least one token)
+    for (int t = blockIdx.x, n = 0; t < b.n_tokens; t += gridDim.x, n = (n + 1) & 31) {
+        if (n == 0) {
+            if (t != (int)blockIdx.x) __syncthreads();               // everybody has read the last of the earlier 32
+            look_up(t);
+            __syncthreads();
+        }
+        float x[NP][4] = {};
+        float2 ss = make_float2(0.f, 0.f);                          // q's and k's sums of squares
+        if (S > 0) {
+#pragma unroll
+            for (int p = 0; p < NP; p++) {
+                if (kind[p] == NONE) continue;
+                const float* f = (const float*)src + (size_t)t * width + from[p];
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                constexpr int W = NP == 1 ? 8 : 4;                  // partial sums in flight together, added in ascending order
+                for (int k = 0; k < S; k += W) {
+                    float4 a[W];
+#pragma unroll
+                    for (int u = 0; u < W; u++) a[u] = *reinterpret_cast<const float4*>(f + (size_t)min(k + u, S - 1) * slice);
+#pragma unroll
+                    for (int u = 0; u < W; u++)
+                        if (k + u < S) { v.x += a[u].x; v.y += a[u].y; v.z += a[u].z; v.w += a[u].w; }
+                }
+                x[p][0] = v.x; x[p][1] = v.y; x[p][2] = v.z; x[p][3] = v.w;
+            }
+        } else {
+#pragma unroll
+            for (int p = 0; p < NP; p++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) x[p][e] = gfb_to_f32(raw[p].v[e]);
+        }
+        if (t + (int)gridDim.x < b.n_tokens) fetch(t + gridDim.x);
+#pragma unroll
+        for (int p = 0; p < NP; p++) {
+            float sum = 0.f;
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                x[p][e] += bi[p][e];
+                sum = fmaf(x[p][e], x[p][e], sum);
+            }
+            ss.x += kind[p] == IS_Q ? sum : 0.f;
+            ss.y += kind[p] == IS_K ? sum : 0.f;
+        }
+        const Place at = places[n];
+        {
+            // two buffers in turn: a warp may write the next token's sums while another still reads this one's
+            const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+            ss.x = gfb_warp_sum(ss.x);
+            ss.y = gfb_warp_sum(ss.y);
+            if (lane == 0) scratch[n & 1][warp] = ss;
+            __syncthreads();
+            ss = lane < nwarp ? scratch[n & 1][lane] : make_float2(0.f, 0.f);
+            ss.x = gfb_warp_sum(ss.x);
+            ss.y = gfb_warp_sum(ss.y);
+        }
+        const float rq = q_norm != nullptr ? 1.0f / sqrtf(ss.x / (float)nq + eps) : 1.f;
+        const float rk = (k_norm != nullptr ? 1.0f / sqrtf(ss.y / (float)max(nk, 1) + eps) : 1.f) * k_scale;
+        if (!at.ok) {                                               // the same for every thread of the block
+            for (int i = threadIdx.x; i < nq; i += blockDim.x) q_out[(size_t)t * nq + i] = gfb_from_f32<T>(0.f);     // q stays defined
+            continue;
+        }
+        const float* cs = table + (size_t)at.pos * rot_dims;         // (not read where rot_dims is 0)
+        T* q_to = q_out + (size_t)t * nq;
+        T* k_to = (T*)kv.k_pool + ((size_t)at.page * G * kv.page_size + at.off) * dk;
+        T* v_to = (T*)kv.v_pool + ((size_t)at.page * G * kv.page_size + at.off) * dv;
+#pragma unroll
+        for (int p = 0; p < NP; p++) {
+            if (kind[p] == NONE) continue;
+            const float r = kind[p] == IS_Q ? rq : kind[p] == IS_K ? rk : 1.f;
+#pragma unroll
+            for (int e = 0; e < 4; e++) x[p][e] *= r * wt[p][e];
 #pragma unroll
             for (int e = 0; e < 4; e += 2)
-                if (j + e < rot_dims) {
-                    const float2 turn = *reinterpret_cast<const float2*>(cs + j + e);
+                if (in_head[p] + e < rot_dims) {
+                    const float2 turn = *reinterpret_cast<const float2*>(cs + in_head[p] + e);
                     const float u = x[p][e], v = x[p][e + 1];
                     x[p][e] = u * turn.x - v * turn.y;
                     x[p][e + 1] = v * turn.x + u * turn.y;
                 }
+            AlignedPack<T, 4> o;
 #pragma unroll
-            for (int e = 0; e < 4; e++) x[p][e] *= f;
+            for (int e = 0; e < 4; e++) o.v[e] = gfb_from_f32<T>(x[p][e]);
+            *reinterpret_cast<AlignedPack<T, 4>*>((kind[p] == IS_Q ? q_to : kind[p] == IS_K ? k_to : v_to) + to[p]) = o;
         }
-        AlignedPack<T, 4> o;
-#pragma unroll
-        for (int e = 0; e < 4; e++) o.v[e] = gfb_from_f32<T>(x[p][e]);
-        *reinterpret_cast<AlignedPack<T, 4>*>(dst) = o;
     }
+}
+
+// how many blocks keep the device full (asked once per kind of kernel and number of threads)
+template <typename T, int NP>
+static int regs_grid(int threads, int n_tokens) {
+    static int resident[33] = {};
+    int& r = resident[threads / 32];
+    if (r == 0) {
+        int per_sm = 0, dev = 0, sms = 0;
+        if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, qkv_prepare_regs_kernel<T, NP>, threads, 0) != cudaSuccess || per_sm < 1) per_sm = 1;
+        if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms < 1) sms = 148;
+        r = per_sm * sms;
+    }
+    return n_tokens < r ? n_tokens : r;
 }
 
 template <typename T, int N, typename... A>
@@ -406,20 +478,20 @@ GFB_API int gfb_qkv_prepare(const void* src, int n_partials, int width, int q_of
     const size_t token_smem = ((size_t)H * dk + (append ? (size_t)G * (dk + dv) : 0)) * sizeof(float);
     if ((norm_opts & NORM_WHOLE) && maps == 1 && !(norm_opts & ~NORM_WHOLE) && token_smem <= 160 * 1024) {
         const bool four = ((q_off | k_off | v_off | width | dk | dv) & 3) == 0
-                          && (((uintptr_t)src | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) == 0;
+                          && (((uintptr_t)src | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)bias | (uintptr_t)q_norm | (uintptr_t)k_norm) & 15) == 0;
         const long cols = (long)H * dk + (append ? (long)G * (dk + dv) : 0);
-        if (four && (table == nullptr || pairing == 0) && cols <= 16384) {
-            // few tokens: as many threads as packs (a token's latency is what counts); many: up to four packs per thread
+        if (four && (table == nullptr || pairing == 0)) {
+            // few tokens: as many threads as packs (a token's latency is what counts); many: a few packs per thread, several tokens per block
             const int packs = (int)(cols / 4);
             const int most = n_tokens <= 128 ? 1024 : 256;
-            int np = (packs + most - 1) / most;
-            np = np <= 1 ? 1 : np <= 2 ? 2 : np <= 4 ? 4 : 8;
+            const int need = (packs + most - 1) / most;
+            const int np = need <= 1 ? 1 : need <= 2 && packs <= 2 * regs_threads(2) ? 2 : 4;
             const int threads = ((packs + np - 1) / np + 31) / 32 * 32;
-            if (threads <= (np == 8 ? 512 : 1024)) {
-#define REGS(T, NP) e = gfb_launch(qkv_prepare_regs_kernel<T, NP>, dim3((unsigned)n_tokens), dim3((unsigned)threads), 0, stream, src, n_partials, slice, width, \
+            if (threads <= regs_threads(np)) {
+#define REGS(T, NP) e = gfb_launch(qkv_prepare_regs_kernel<T, NP>, dim3((unsigned)regs_grid<T, NP>(threads, n_tokens)), dim3((unsigned)threads), 0, stream, src, n_partials, slice, width, \
                                    q_off, k_off, v_off, bias, b_dt, (T*)q_out, kv, b, table, table_len, table != nullptr ? rot_dims : 0, q_norm, k_norm, w_dt, eps, \
                                    k_scale, H, G, dk, dv, append, status)
-#define REGS_NP(T) do { if (np == 1) REGS(T, 1); else if (np == 2) REGS(T, 2); else if (np == 4) REGS(T, 4); else REGS(T, 8); } while (0)
+#define REGS_NP(T) do { if (np == 1) REGS(T, 1); else if (np == 2) REGS(T, 2); else REGS(T, 4); } while (0)
                 if (dt == GFB_BF16) REGS_NP(__nv_bfloat16);
                 else if (dt == GFB_F32) REGS_NP(float);
                 else return gfb_fail("gfb_qkv_prepare: unknown type %d", dt);

@@ -8,6 +8,8 @@ the small, self-ending workload that profiler captures are taken on.
     python -m gpt_fast_b200.engine.kernel_bench attention --batch 1 --context 0 --new 2048
     python -m gpt_fast_b200.engine.kernel_bench sample --batch 8 --vocab 128256
     python -m gpt_fast_b200.engine.kernel_bench experts --tokens 2048 --experts 16 --top 4 --ff 1792 --dim 2048
+    python -m gpt_fast_b200.engine.kernel_bench streams --rows 2048 --dim 2048 --streams 4
+    python -m gpt_fast_b200.engine.kernel_bench qkv --rows 2048 --heads 16 --kv_heads 4 --head_dim 128
     python -m gpt_fast_b200.engine.kernel_bench gla --tokens 2048 --heads 16 --head_dim 128 --v_dim 128
 
 Weights are cycled through enough copies to exceed the L2 cache, so a memory-
@@ -185,6 +187,40 @@ def bench_gla(a):
     ops.check_status(meta.status)
 
 
+def bench_streams(a):
+    """Several residual streams: a sublayer's output (a tensor, or partial sums) goes into them and the next input comes out normed.
+    Enough copies of everything are cycled through to exceed the L2 cache."""
+    T, D, n = a.rows, a.dim, a.streams
+    nbytes = T * D * (4 * (2 * n + max(a.partials, 1)) + 2)
+    copies = max(1, min(64, int(3 * L2_BYTES // nbytes) + 1))
+    xs = [torch.randn(n, T, D, device="cuda") for _ in range(copies)]
+    ys = [torch.randn(a.partials, T, D, device="cuda") if a.partials else torch.randn(T, D, device="cuda") for _ in range(copies)]
+    mix, leave, enter = torch.eye(n, device="cuda"), torch.ones(n, device="cuda") * 1e-3, torch.full((n,), 1.0 / n, device="cuda")
+    w, out = torch.ones(D, device="cuda", dtype=torch.bfloat16), [torch.empty(T, D, device="cuda", dtype=torch.bfloat16) for _ in range(copies)]
+    us = graph_time_us(lambda i: ops.streams(xs[i % copies], n, False, xs[i % copies], mix, leave, [ys[i % copies]], enter, w, 1e-5, out[i % copies]), a.reps)
+    print(f"streams rows={T} dim={D} streams={n} partial sums={a.partials}: {us:.1f} us, {nbytes / us / 1e3:.0f} GB/s")
+
+
+def bench_qkv(a):
+    """q, k and v of `rows` tokens with biases and a norm over the whole projection into queries and cache."""
+    H, G, d, T = a.heads, a.kv_heads, a.head_dim, a.rows
+    W = (H + 2 * G) * d
+    new = T // a.batch
+    meta, kv = paged_batch(a.batch, 512, new, G, d)
+    nbytes = T * W * (2 + (4 * a.partials if a.partials else 2))
+    copies = max(1, min(64, int(3 * L2_BYTES // nbytes) + 1))
+    srcs = [torch.randn(T, W, device="cuda").bfloat16() for _ in range(copies)]
+    parts = [torch.randn(a.partials, T, W, device="cuda") for _ in range(copies)] if a.partials else [None] * copies
+    q = torch.empty(T, H, d, device="cuda", dtype=torch.bfloat16)
+    table = torch.empty(512 + new + 64, a.rot // 2, 2, device="cuda")
+    ops.rope_table((1.0 / (10000 ** (torch.arange(a.rot // 2).float() * 2 / a.rot))).cuda(), table)
+    bias, qn, kn = torch.randn(W, device="cuda"), torch.ones(H * d, device="cuda").bfloat16(), torch.ones(G * d, device="cuda").bfloat16()
+    us = graph_time_us(lambda i: ops.qkv_prepare(srcs[i % copies], parts[i % copies], (0, H * d, (H + G) * d), q, kv, meta, H, G, d, d, table=table,
+                                                 rot_dims=a.rot, pairing=a.pairing, q_norm=qn, k_norm=kn, norm_eps=1e-5, norm_whole=True, bias=bias), a.reps)
+    print(f"qkv rows={T} heads={H}/{G} of {d} pairs={a.pairing} partial sums={a.partials}: {us:.1f} us, {nbytes / us / 1e3:.0f} GB/s")
+    ops.check_status(meta.status)
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser(prog="kernel_bench")
     sub = ap.add_subparsers(dest="what", required=True)
@@ -214,12 +250,21 @@ def main(argv=None):
     p.add_argument("--top", type=int, default=4); p.add_argument("--ff", type=int, default=1792)
     p.add_argument("--dim", type=int, default=2048); p.add_argument("--limit", type=float, default=7.0)
     p.add_argument("--reps", type=int, default=5)
+    p = sub.add_parser("streams")
+    p.add_argument("--rows", type=int, default=2048); p.add_argument("--dim", type=int, default=2048)
+    p.add_argument("--streams", type=int, default=4); p.add_argument("--partials", type=int, default=0)
+    p.add_argument("--reps", type=int, default=20)
+    p = sub.add_parser("qkv")
+    p.add_argument("--rows", type=int, default=2048); p.add_argument("--batch", type=int, default=1); p.add_argument("--heads", type=int, default=16)
+    p.add_argument("--kv_heads", type=int, default=4); p.add_argument("--head_dim", type=int, default=128)
+    p.add_argument("--rot", type=int, default=64); p.add_argument("--partials", type=int, default=0)
+    p.add_argument("--pairing", default="interleaved", choices=["interleaved", "half"]); p.add_argument("--reps", type=int, default=20)
     p = sub.add_parser("gla")
     p.add_argument("--batch", type=int, default=1); p.add_argument("--tokens", type=int, default=2048)
     p.add_argument("--heads", type=int, default=16); p.add_argument("--head_dim", type=int, default=128)
     p.add_argument("--v_dim", type=int, default=128); p.add_argument("--reps", type=int, default=10)
     a = ap.parse_args(argv)
-    {"gla": bench_gla, "experts": bench_experts, "linear": bench_linear, "attention": bench_attention, "sample": bench_sample, "norm": bench_norm}[a.what](a)
+    {"gla": bench_gla, "streams": bench_streams, "qkv": bench_qkv, "experts": bench_experts, "linear": bench_linear, "attention": bench_attention, "sample": bench_sample, "norm": bench_norm}[a.what](a)
     ops.check_status(ops.new_status("cuda"))
     return 0
 
